@@ -23,13 +23,14 @@ from typing import Optional, Sequence
 
 @dataclass(frozen=True)
 class RopeScalingSpec:
-    """Frequency-dependent scaling of rotary frequencies ("llama3" rule)."""
+    """Scaling of rotary frequencies: "llama3" (frequency-dependent) or "linear" (every
+    frequency divided by ``factor``; the other fields are not read)."""
 
     rope_type: str
     factor: float
-    low_freq_factor: float
-    high_freq_factor: float
-    original_max_position_embeddings: int
+    low_freq_factor: float = 1.0
+    high_freq_factor: float = 1.0
+    original_max_position_embeddings: int = 0
 
 
 @dataclass(frozen=True)
@@ -86,6 +87,10 @@ class AttentionSpec:
     + 1) / every) + 1)``.  ``softcap``: scores become ``softcap * tanh(score / softcap)`` after
     the scale.  ``sink``: "learned" puts ``exp(sink_h)``, a parameter a head, into the
     softmax's denominator (it has no key and no value); "zero" puts exp(0) = 1 there.
+    ``chunk``: a token at position p sees keys of its own chunk only, ``(p // chunk) * chunk ..
+    p``, chunks counted from the sequence's start.  ``weights``: "softmax", or "sigmoid": the
+    weight of a visible key is ``sigmoid(score)``, nothing is normalised over the keys.
+    ``score_bias``: a learned number a head is added to the (scaled, capped) scores.
     """
 
     kind: str = "attention"
@@ -109,6 +114,9 @@ class AttentionSpec:
     q_temp: Optional[tuple] = None
     softcap: Optional[float] = None
     sink: Optional[str] = None
+    chunk: Optional[int] = None
+    weights: str = "softmax"
+    score_bias: bool = False
 
     @property
     def value_dim(self) -> int:
@@ -120,7 +128,8 @@ class AttentionSpec:
         return (not self.keep_first and self.v_head_dim in (None, self.head_dim)
                 and not self.bias and self.qk_norm_eps is None and self.conv_taps == 0
                 and not self.value_from_key and not self.head_gate and not self.feature_gate
-                and self.q_temp is None and self.softcap is None and self.sink is None)
+                and self.q_temp is None and self.softcap is None and self.sink is None
+                and self.chunk is None and self.weights == "softmax" and not self.score_bias)
 
 
 @dataclass(frozen=True)
@@ -215,6 +224,64 @@ class GatedDeltaSpec:
 
 
 @dataclass(frozen=True)
+class TimeMixingSpec:
+    """kind "time_mixing": RWKV-style time mixing, a matrix memory per head with a decay per
+    key channel and a bonus for the current token, carried as per-request state.
+
+    With h' the previous token's input (zeros at the start), each of r, k, v, g and w reads a
+    mix of its own, ``h + (h' - h) * mu``; r, k, v (``num_heads`` heads of ``dim``) and the gate
+    ``silu(g)`` are projections of theirs; ``decay = exp(-exp(W_w2 tanh(W_w1 mix_w) + w0))`` per
+    head and key channel (W_w1 has ``decay_rank`` rows).  Per head: ``o = (S + diag(u) k v^T)^T
+    r``, then ``S = diag(decay) S + k v^T``.  Each head's o is divided by its root mean square
+    (``norm_eps``); the heads are scaled by a weight a feature, gated and projected back.  S
+    (float) and the last input row are per-request state.
+    """
+
+    kind: str = "time_mixing"
+    hidden_size: int = 0
+    num_heads: int = 0
+    dim: int = 0
+    decay_rank: int = 0
+    norm_eps: float = 1e-6
+    shares_kv: bool = False
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """kind "state_space": the Mamba-2 mixer, a matrix state [state, v_dim] per head with one
+    decay a head, carried as per-request state.
+
+    ``W_in h = [z: inner | x: inner | B: groups * state | C: groups * state | dt: heads]``, inner =
+    ``num_heads * v_dim``; x, B and C pass a causal convolution of ``conv`` taps per channel with
+    a bias, and SiLU; ``dt = softplus(dt + dt_bias)``.  Head h reads B and C of group ``h //
+    (num_heads / groups)``: ``S = exp(-exp(A_log) dt) S + dt B x^T``, ``y = S^T C + D x``.  y is
+    multiplied by ``silu(z)``, divided by its root mean square in ``norm_groups`` equal parts
+    (``norm_eps``), scaled and projected back.  S (float) and the convolution's last ``conv -
+    1`` inputs are per-request state.
+    """
+
+    kind: str = "state_space"
+    hidden_size: int = 0
+    num_heads: int = 0
+    v_dim: int = 0
+    state: int = 0
+    groups: int = 1
+    conv: int = 1
+    norm_groups: int = 1
+    norm_eps: float = 1e-6
+    shares_kv: bool = False
+
+    @property
+    def inner(self) -> int:
+        return self.num_heads * self.v_dim
+
+    @property
+    def channels(self) -> int:
+        """What the convolution runs over: x, B and C."""
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass(frozen=True)
 class MatrixMemorySpec:
     """kind "mlstm": a matrix memory per head (the mLSTM cell of xLSTM), carried from token
     to token as per-request state instead of a key/value cache.
@@ -285,6 +352,10 @@ class RoutedExpertsSpec:
     choice only (the weights use the scores without it).  ``identity_experts``: the router
     has that many further outputs, standing for experts without tensors whose output is
     their input.
+    ``activation`` "clamped_swish" (gated): with ``g = min(gate u, limit)`` and ``v = clamp(up u,
+    -limit, limit)`` the hidden units are ``g sigmoid(swish_alpha g) (v + 1)``; the shared expert
+    clamps at ``shared_limit``.  ``shared_gate``: the shared expert's output is multiplied by
+    ``sigmoid(w_sg x)``, one number a token.
     """
 
     kind: str = "routed_experts"
@@ -300,6 +371,10 @@ class RoutedExpertsSpec:
     gated: bool = True
     choice_bias: bool = False
     identity_experts: int = 0
+    limit: float = 0.0
+    shared_limit: float = 0.0
+    swish_alpha: float = 1.702
+    shared_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -340,6 +415,9 @@ class BlockSpec:
     residual_mult * out_q[t] * y``; the model's residual is the sum of the copies.  ``streams``
     0 is the plain ``x += residual_mult * sublayer(norm(x))`` through the same kernels.
     ``ffn`` None leaves the second sublayer out.
+    kind "side_by_side": ``h += mixer(n~) + ffn(n)`` with one norm, ``n = norm1(h)`` (``norm2`` is
+    None); with ``token_shift`` the mixer reads ``n~ = n + (n' - n) * shift``, n' the previous
+    token's n (zeros at the start; the last n of a sequence is per-request state), else n.
     ``mixer`` / ``ffn`` are any registered spec; they may differ from block
     to block within one model.
     """
@@ -353,6 +431,7 @@ class BlockSpec:
     norm2_post: Optional[NormSpec] = None
     residual_mult: float = 1.0
     streams: int = 0
+    token_shift: bool = False
 
 
 @dataclass(frozen=True)
@@ -362,11 +441,22 @@ class RunEntry:
     ``block``: index into ``ModelLayout.blocks`` (a block may appear twice,
     its weights are then shared).  ``cache``: index of the cache this run
     reads and writes; by default every run has its own.  A run whose mixer
-    ``shares_kv`` names the cache of the earlier run it reads.
+    ``shares_kv`` names the cache of the earlier run it reads.  ``loop_input``: before this
+    run the residual goes through the layout's ``loop_input`` part (the first run of each
+    pass of a looped stretch).
     """
 
     block: int
     cache: int
+    loop_input: bool = False
+
+
+@dataclass(frozen=True)
+class LoopInputSpec:
+    """kind "concat_linear": the residual x becomes ``W [x; x0]``, x0 the embedding output."""
+
+    kind: str = "concat_linear"
+    hidden_size: int = 0
 
 
 @dataclass(frozen=True)
@@ -383,6 +473,8 @@ class ModelLayout:
     # table and a plain linear head of the layout's sizes
     embedding: Optional[object] = None
     head: Optional[object] = None
+    # what the residual passes before a run order entry with ``loop_input``
+    loop_input: Optional[object] = None
 
     def embedding_spec(self):
         return self.embedding or EmbeddingSpec(vocab_size=self.vocab_size,
@@ -402,6 +494,9 @@ class ModelLayout:
             if not 0 <= entry.block < len(self.blocks):
                 raise ValueError(f"run order entry {pos} names block {entry.block}, "
                                  f"but the layout has {len(self.blocks)} blocks")
+            if entry.loop_input and self.loop_input is None:
+                raise ValueError(f"run order entry {pos} asks for a loop input, but the layout "
+                                 "has none")
             mixer = self.blocks[entry.block].mixer
             if getattr(mixer, "shares_kv", False):
                 if entry.cache not in owners:

@@ -108,3 +108,8 @@ def _register_builtin() -> None:
 
     if "Mokotar" not in _ARCHITECTURES:
         register_architecture("Mokotar", MokotarConfig, mokotar_checkpoint_map)
+    from ..weights.sokalorn import sokalorn_checkpoint_map
+    from .sokalorn import SokalornConfig
+
+    if "Sokalorn" not in _ARCHITECTURES:
+        register_architecture("Sokalorn", SokalornConfig, sokalorn_checkpoint_map)

@@ -21,7 +21,10 @@
 //             them, scores q.k * scale, float statistics and sums.  With `softcap` > 0 a
 //             score becomes softcap * tanh(score / softcap); with `sink` the denominator of
 //             head h also holds exp(sink[h]), which has no key and no value; a gate per
-//             feature multiplies the output by sigmoid(gate[t][h * vd + d]).
+//             feature multiplies the output by sigmoid(gate[t][h * vd + d]).  With `chunk` > 0 the
+//             window is the token's chunk instead: lo = p / chunk * chunk.  `bias` adds a number
+//             a head to the (scaled, capped) scores; with `sigmoid` a visible key's weight is
+//             sigmoid(score) and nothing is normalised over the keys.
 //
 // A cache page is [nkv][page_size][hd] keys followed by [nkv][page_size][vd] values.
 // Norms, angles, scores, probabilities and output sums are float for both activation types.
@@ -299,6 +302,9 @@ struct SinkArgs {
     const float* sink;          // null, or one number a query head
     const float* gate;          // null, or float rows with a number per (head, feature)
     int gate_stride;
+    int chunk;                  // 0: none
+    int sigmoid;                // 1: weights are sigmoids of the scores
+    const float* bias;          // null, or one number a query head, added to the scores
 };
 
 // The v-th key a token sees: the kept first keys come before the window's.
@@ -332,7 +338,8 @@ sink_attention_generic_kernel(const A* __restrict__ q, A* __restrict__ out,
     kv_cache = pdl_after(kv_cache, waited);
     const float* gate = pdl_after(a.gate, waited);
     const int hi = cache_pos[t] + 1;
-    const int lo = (a.window > 0 && hi > a.window) ? hi - a.window : 0;
+    const int lo = a.chunk > 0 ? (hi - 1) / a.chunk * a.chunk
+                               : ((a.window > 0 && hi > a.window) ? hi - a.window : 0);
     const int kept = a.keep_first < lo ? a.keep_first : lo;
     const int visible = kept + hi - lo;
     const int* bt = block_table + (size_t)token_req[t] * a.bt_stride;
@@ -375,12 +382,18 @@ sink_attention_generic_kernel(const A* __restrict__ q, A* __restrict__ out,
                 for (int d = 0; d < hd; ++d) dot = fmaf(qv[d], kv[d], dot);
                 s = dot * a.scale;
                 if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+                if (a.bias != nullptr) s += a.bias[kvh * G + g];
             }
             sc[idx] = s;
         }
         __syncthreads();
         for (int g = warp; g < G; g += SA_THREADS / 32) {
             const float s = sc[g * SA_TILE + lane];
+            if (a.sigmoid) {                   // (a masked key's score is -inf: weight 0)
+                sc[g * SA_TILE + lane] = 1.f / (1.f + expf(-s));
+                if (lane == 0) alpha_s[g] = 1.f;
+                continue;
+            }
             const float m_old = m_s[g];
             const float m_new = fmaxf(m_old, warp_max(s));  // the tile's first key is visible
             const float p = expf(s - m_new);
@@ -430,7 +443,7 @@ sink_attention_generic_kernel(const A* __restrict__ q, A* __restrict__ out,
     for (int k = 0; k < SA_MAX_ACC; ++k) {
         const int o = tid + k * SA_THREADS;
         if (o < n_out) {
-            float r = acc[k] / l_s[o / vd];
+            float r = a.sigmoid ? acc[k] : acc[k] / l_s[o / vd];
             if (gate != nullptr)
                 r /= 1.f + expf(-gate[(size_t)t * a.gate_stride + (size_t)kvh * G * vd + o]);
             orow[o] = from_float<A>(r);
@@ -447,8 +460,10 @@ MSTAR_API int mstar_sink_attention_generic(const void* q, int q_stride, void* ou
                                            int hd, int vd, int page_size, int window,
                                            int keep_first, float scale, int act_dtype,
                                            float softcap, const float* sink, const float* gate,
-                                           int gate_stride, void* stream) {
+                                           int gate_stride, int chunk, int sigmoid,
+                                           const float* bias, void* stream) {
     if (tokens <= 0) return 0;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sigmoid && sink != nullptr)) return -1;
     if (nkv <= 0 || nq % nkv != 0 || hd <= 0 || vd <= 0) return -1;
     const int G = nq / nkv;
     if (G * vd > SA_MAX_ACC * SA_THREADS) return -1;
@@ -458,7 +473,7 @@ MSTAR_API int mstar_sink_attention_generic(const void* q, int q_stride, void* ou
     if (smem > 200 * 1024) return -1;
     cudaStream_t s = (cudaStream_t)stream;
     SinkArgs a{nq, nkv, hd, vd, page_size, bt_stride, window, keep_first, q_stride, scale,
-               softcap, sink, gate, gate_stride};
+               softcap, sink, gate, gate_stride, chunk, sigmoid, bias};
     dim3 grid(tokens, nkv);
     static size_t configured_f32 = 0, configured_bf16 = 0;
     if (act_dtype == MSTAR_F32) {

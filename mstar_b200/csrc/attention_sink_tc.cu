@@ -15,7 +15,10 @@
 // Options: a soft cap (a score becomes cap * tanh(score / cap) after the scale), a sink a
 // query head (exp(sink_h) joins the softmax's denominator where a row's last partial sums
 // meet; it has no key and no value), and a gate on the output, one number a head or one a
-// feature.
+// feature.  With `chunk` a row's window is its chunk of positions; with `bias` a number a head is
+// added to the capped scores; the SIGMOID form weights a visible key by the sigmoid of its score:
+// no maximum, no sum, no rescaling, and the partial sums of warps and splits simply add up (they
+// carry the maximum 0, and the sum 1 in one of them, so that the merges need no form of their own).
 //
 // With few rows (decoding) the visited keys are shared among `splits` CTAs, each leaving an
 // unnormalised partial (o, running maximum, sum) in scratch, and a second kernel merges.
@@ -44,6 +47,8 @@ struct SinkTcArgs {
     float scale, softcap;       // softcap 0: none
     float cap_in, cap_log2e;    // 2 log2(e) scale / softcap and softcap log2(e)
     const float* sink;          // null, or one number a query head
+    int chunk;                  // 0: none
+    const float* bias;          // null, or one number a query head
 };
 
 __device__ __forceinline__ float st_head_gate(const float* gate, int stride, int tok, int head) {
@@ -69,7 +74,7 @@ template <int D> __device__ __forceinline__ int st_off(int row, int c) { return 
 // and each a quarter of every key tile (keys 16 w .. 16 w + 15 of the tile), with a running
 // maximum, sum and output of its own; the four are merged through shared memory at the end.
 // One warp alone would issue a tile's products one after the other while three wait.
-template <int D, int NSTAGE, bool KEYSPLIT>
+template <int D, int NSTAGE, bool KEYSPLIT, bool SIGMOID>
 __global__ void __launch_bounds__(ST_THREADS)
 sink_attention_tc_kernel(SinkTcArgs a) {
     constexpr int CPR = D / 8;
@@ -96,7 +101,9 @@ sink_attention_tc_kernel(SinkTcArgs a) {
     const int W = a.window > 0 ? a.window : 0x3fffffff;
     const int last_row = min(rows_total, row0 + ST_ROWS) - 1;
     const int hi = past + last_row / G + 1;
-    const int lo = max(0, past + row0 / G - W + 1);
+    // the oldest key that the window (or chunk) of a cache position holds
+    auto window_lo = [&](int cp) { return a.chunk > 0 ? cp / a.chunk * a.chunk : max(0, cp - W + 1); };
+    const int lo = window_lo(past + row0 / G);
     const int kept = min(a.keep_first, lo);    // kept first keys before the CTA's window
     const int visible = kept + hi - lo;
 
@@ -146,7 +153,13 @@ sink_attention_tc_kernel(SinkTcArgs a) {
     const int cpB = past + min(rowB, rows_total - 1) / G;
     // the warp's rows together: newest key any row sees, oldest window key any row sees
     const int warp_hi = past + min(row0 + wrow + 15, rows_total - 1) / G;
-    const int warp_lo = max(0, past + min(row0 + wrow, rows_total - 1) / G - W + 1);
+    const int warp_lo = window_lo(past + min(row0 + wrow, rows_total - 1) / G);
+    const int loA = window_lo(cpA), loB = window_lo(cpB);
+    float biasA = 0.f, biasB = 0.f;            // base-2 domain
+    if (a.bias != nullptr) {
+        biasA = a.bias[kvh * G + min(rowA, rows_total - 1) % G] * 1.4426950408889634f;
+        biasB = a.bias[kvh * G + min(rowB, rows_total - 1) % G] * 1.4426950408889634f;
+    }
 
     float o[D / 8][4];
 #pragma unroll
@@ -204,7 +217,8 @@ sink_attention_tc_kernel(SinkTcArgs a) {
                     const int key = v < kept ? v : lo + v - kept;
                     const bool upper = q4 < 2;
                     const int cp = upper ? cpA : cpB;
-                    const bool ok = v < visible && key <= cp && (cp - key < W || key < a.keep_first);
+                    const bool ok = v < visible && key <= cp &&
+                                    (key >= (upper ? loA : loB) || key < a.keep_first);
                     float sv = -INFINITY;
                     if (ok) {
                         // cap * tanh(x / cap) * log2(e) with tanh(z) = 1 - 2 / (2^(2 z log2 e) + 1):
@@ -212,10 +226,16 @@ sink_attention_tc_kernel(SinkTcArgs a) {
                         sv = a.softcap > 0.f
                                  ? a.cap_log2e * (1.f - __fdividef(2.f, exp2f(s[j][q4] * a.cap_in) + 1.f))
                                  : s[j][q4] * a.scale_log2e;
+                        sv += upper ? biasA : biasB;
+                    }
+                    if constexpr (SIGMOID) {   // (a masked key's score is -inf: weight 0)
+                        s[j][q4] = __fdividef(1.f, 1.f + exp2f(-sv));
+                        continue;
                     }
                     s[j][q4] = sv;
                     if (upper) mx0 = fmaxf(mx0, sv); else mx1 = fmaxf(mx1, sv);
                 }
+            if constexpr (!SIGMOID) {
             mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
             mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
             mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
@@ -240,6 +260,7 @@ sink_attention_tc_kernel(SinkTcArgs a) {
 #pragma unroll
             for (int n = 0; n < D / 8; ++n) {
                 o[n][0] *= al0; o[n][1] *= al0; o[n][2] *= al1; o[n][3] *= al1;
+            }
             }
             // O += P V with P = P1 + P2 + P3, three bfloat16 parts that hold the float exactly.
             // A block of 16 keys at a time: its three parts of P, then every value fragment
@@ -290,6 +311,10 @@ sink_attention_tc_kernel(SinkTcArgs a) {
     l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    if constexpr (SIGMOID) {
+        m0 = m1 = 0.f;
+        l0 = l1 = (split == 0 && (!KEYSPLIT || warp == 0)) ? 1.f : 0.f;
+    }
     if constexpr (KEYSPLIT) {
         // the four warps' partials of rows 0..15 meet in shared memory (the key/value stages are
         // done with): [warp][row][vd + 2] floats, then every thread sums a share of (row, feature)
@@ -428,12 +453,12 @@ __global__ void sink_merge_kernel(const float* __restrict__ scratch, bf16* __res
     }
 }
 
-template <int D, int NSTAGE, bool KEYSPLIT>
+template <int D, int NSTAGE, bool KEYSPLIT, bool SIGMOID>
 static int launch_sink_tc_stages(const SinkTcArgs& a, int entries, int max_q_len, cudaStream_t s) {
     const size_t smem = (size_t)(2 * NSTAGE + 1) * ST_TILE * (D + 8) * sizeof(bf16);
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(sink_attention_tc_kernel<D, NSTAGE, KEYSPLIT>,
+        cudaError_t e = cudaFuncSetAttribute(sink_attention_tc_kernel<D, NSTAGE, KEYSPLIT, SIGMOID>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
@@ -442,21 +467,21 @@ static int launch_sink_tc_stages(const SinkTcArgs& a, int entries, int max_q_len
     const long long tiles = ((long long)max_q_len * G + ST_ROWS - 1) / ST_ROWS;
     if (tiles * a.splits > 2147483647LL) return -1;
     dim3 grid((unsigned)(tiles * a.splits), a.nkv, entries);
-    mstar_launch((sink_attention_tc_kernel<D, NSTAGE, KEYSPLIT>), grid, dim3(ST_THREADS), smem, s, a);
+    mstar_launch((sink_attention_tc_kernel<D, NSTAGE, KEYSPLIT, SIGMOID>), grid, dim3(ST_THREADS), smem, s, a);
     return launch_status();
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 static int launch_sink_tc(const SinkTcArgs& a, int entries, int max_q_len, cudaStream_t s) {
     // one row tile per (entry, kv head): few rows, deep prefetch (where shared memory has room)
     const long long rows = (long long)max_q_len * (a.nq / a.nkv);
     if constexpr (D <= 128) {
-        if (rows <= 16) return launch_sink_tc_stages<D, 4, true>(a, entries, max_q_len, s);
-        if (rows <= ST_ROWS) return launch_sink_tc_stages<D, 4, false>(a, entries, max_q_len, s);
+        if (rows <= 16) return launch_sink_tc_stages<D, 4, true, SIGMOID>(a, entries, max_q_len, s);
+        if (rows <= ST_ROWS) return launch_sink_tc_stages<D, 4, false, SIGMOID>(a, entries, max_q_len, s);
     } else {
-        if (rows <= 16) return launch_sink_tc_stages<D, 2, true>(a, entries, max_q_len, s);
+        if (rows <= 16) return launch_sink_tc_stages<D, 2, true, SIGMOID>(a, entries, max_q_len, s);
     }
-    return launch_sink_tc_stages<D, 2, false>(a, entries, max_q_len, s);
+    return launch_sink_tc_stages<D, 2, false, SIGMOID>(a, entries, max_q_len, s);
 }
 
 // Entries [0, entries) of the batch; q: [tokens] rows of q_stride elements; out: [tokens,
@@ -470,7 +495,9 @@ MSTAR_API int mstar_sink_attention_tc(const void* q, int q_stride, void* out, co
                                       int nq, int nkv, int hd, int vd, int page_size, int window,
                                       int keep_first, float scale, int splits, float* scratch,
                                       const float* gate, int gate_stride, int gate_features,
-                                      float softcap, const float* sink, void* stream) {
+                                      float softcap, const float* sink, int chunk, int sigmoid,
+                                      const float* bias, void* stream) {
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sigmoid && sink != nullptr)) return -1;
     if (entries <= 0 || max_q_len <= 0) return 0;
     if (nkv <= 0 || nq % nkv != 0 || entries > 65535 || nkv > 65535) return -1;
     if (hd % 8 || vd % 8 || hd <= 0 || vd <= 0 || hd > 256 || vd > 256 || splits < 1 || splits > 64)
@@ -503,14 +530,20 @@ MSTAR_API int mstar_sink_attention_tc(const void* q, int q_stride, void* out, co
     a.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
     a.cap_log2e = softcap * 1.4426950408889634f;
     a.sink = sink;
+    a.chunk = chunk;
+    a.bias = bias;
     cudaStream_t s = (cudaStream_t)stream;
     const int wide = hd > vd ? hd : vd;
     int code;
-    if (wide <= 32) code = launch_sink_tc<32>(a, entries, max_q_len, s);
-    else if (wide <= 64) code = launch_sink_tc<64>(a, entries, max_q_len, s);
-    else if (wide <= 96) code = launch_sink_tc<96>(a, entries, max_q_len, s);
-    else if (wide <= 128) code = launch_sink_tc<128>(a, entries, max_q_len, s);
-    else code = launch_sink_tc<256>(a, entries, max_q_len, s);
+#define GO(D)                                                                                     \
+    (sigmoid ? launch_sink_tc<D, true>(a, entries, max_q_len, s)                                  \
+             : launch_sink_tc<D, false>(a, entries, max_q_len, s))
+    if (wide <= 32) code = GO(32);
+    else if (wide <= 64) code = GO(64);
+    else if (wide <= 96) code = GO(96);
+    else if (wide <= 128) code = GO(128);
+    else code = GO(256);
+#undef GO
     if (code != 0 || splits == 1) return code;
     const int rows = tokens * nq;
     mstar_launch(sink_merge_kernel, dim3((rows + 3) / 4), dim3(128), 0, s, (const float*)scratch,

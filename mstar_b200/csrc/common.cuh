@@ -65,6 +65,13 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// The clamped gate of a gated feed-forward: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g sigmoid(alpha g) (u + 1).
+__device__ __forceinline__ float clamped_swish(float gate, float up, float limit, float alpha) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+
 // Sum over a whole block; `scratch` holds at least 32 floats of shared memory.
 // Every thread gets the result.  Safe to call repeatedly with the same scratch.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {

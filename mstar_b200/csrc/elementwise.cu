@@ -245,7 +245,8 @@ MSTAR_API int mstar_gather_add_rows(const float* resid, const void* delta, int a
 // gate_up: [rows, 2*inter] with gate first (mstar/model/components/distributed/
 // mlp.py:78-81); out: [rows, inter].  silu(x) = x / (1 + exp(-x)), or the tanh form of gelu,
 // in float.
-// kind 0: relu(x)^2, 1: gelu (tanh form), 2: silu.
+// kind 0: relu(x)^2, 1: gelu (tanh form), 2: silu.  The gated kernel also takes 3: the clamped
+// swish of common.cuh with its limit and alpha.
 __device__ __forceinline__ float plain_activation(float v, int kind) {
     if (kind == 0) {
         const float r = fmaxf(v, 0.f);
@@ -258,7 +259,7 @@ __device__ __forceinline__ float plain_activation(float v, int kind) {
 
 template <typename A>
 __global__ void silu_mul_kernel(const A* __restrict__ gate_up, A* __restrict__ out, int inter,
-                                size_t total, int kind) {
+                                size_t total, int kind, float limit, float alpha) {
     gate_up = pdl_after(gate_up, pdl_wait());
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
          idx += (size_t)gridDim.x * blockDim.x) {
@@ -267,24 +268,25 @@ __global__ void silu_mul_kernel(const A* __restrict__ gate_up, A* __restrict__ o
         const A* p = gate_up + row * 2 * (size_t)inter;
         const float g = to_float(p[col]);
         const float u = to_float(p[inter + col]);
-        out[idx] = from_float<A>(plain_activation(g, kind) * u);
+        out[idx] = from_float<A>(kind == 3 ? clamped_swish(g, u, limit, alpha)
+                                           : plain_activation(g, kind) * u);
     }
 }
 
 MSTAR_API int mstar_silu_mul(const void* gate_up, void* out, int act_dtype, int rows, int inter,
-                             int kind, void* stream) {
+                             int kind, float limit, float alpha, void* stream) {
     const size_t total = (size_t)rows * inter;
     if (total == 0) return 0;
-    if (kind != 1 && kind != 2) return -1;
+    if (kind < 1 || kind > 3) return -1;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = 256;
     size_t blocks = (total + threads - 1) / threads;
     const size_t most = (size_t)device_sm_count() * 32;   // a grid-stride loop takes the rest
     if (blocks > most) blocks = most;
     if (act_dtype == MSTAR_F32)
-        mstar_launch((silu_mul_kernel<float>), dim3((int)blocks), dim3(threads), 0, s, (const float*)gate_up, (float*)out, inter, total, kind);
+        mstar_launch((silu_mul_kernel<float>), dim3((int)blocks), dim3(threads), 0, s, (const float*)gate_up, (float*)out, inter, total, kind, limit, alpha);
     else
-        mstar_launch((silu_mul_kernel<bf16>), dim3((int)blocks), dim3(threads), 0, s, (const bf16*)gate_up, (bf16*)out, inter, total, kind);
+        mstar_launch((silu_mul_kernel<bf16>), dim3((int)blocks), dim3(threads), 0, s, (const bf16*)gate_up, (bf16*)out, inter, total, kind, limit, alpha);
     return launch_status();
 }
 

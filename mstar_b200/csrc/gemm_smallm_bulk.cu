@@ -80,8 +80,14 @@ struct SbRope {
     int nq, nkv, hd, page_size, bt_stride;
     // plain form: 1 squares the positive part of every sum before it is stored (a
     // feed-forward's first product with its relu-squared, as one kernel); gated form: 0 gates
-    // by the SiLU, 2 by the tanh form of gelu
+    // by the SiLU, 2 by the tanh form of gelu, 3 by the clamped swish with limit and alpha
     int act;
+    float limit, alpha;
+    // plain form with plane_rows > 0: output features [p plane_rows, (p + 1) plane_rows) are
+    // products with the rows of plane p of x, plane_stride elements apart (the last plane, planes
+    // - 1, takes what is left)
+    int plane_rows, planes;
+    long long plane_stride;
 };
 
 __host__ __device__ constexpr int sb_rows(bool gated, int nt) { return (gated ? 16 : 8) * nt; }
@@ -179,14 +185,17 @@ smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT*
     const bf16* xb = x + (size_t)min(g + 8, M - 1) * ldx + 8 * t;
     // this warp's blocks of a chunk: warp, warp + 8, ...  (at most 4 of 32)
     constexpr int PER = SB_KC / 32 / SB_WARPS;
-    auto load_x = [&](int ch, uint4 (&xv)[PER], uint4 (&xw)[PER]) {
+    auto load_x = [&](int strip, int ch, uint4 (&xv)[PER], uint4 (&xw)[PER]) {
+        size_t plane = 0;
+        if (MODE == SB_PLAIN && rp.plane_rows > 0)
+            plane = (size_t)min(strip * 8 * NT / rp.plane_rows, rp.planes - 1) * rp.plane_stride;
 #pragma unroll
         for (int u = 0; u < PER; ++u) {
             const int k = ch * SB_KC + (warp + u * SB_WARPS) * 32;
             xv[u] = xw[u] = make_uint4(0u, 0u, 0u, 0u);
             if (k < K) {
-                xv[u] = *reinterpret_cast<const uint4*>(xa + k);
-                if (M16) xw[u] = *reinterpret_cast<const uint4*>(xb + k);
+                xv[u] = *reinterpret_cast<const uint4*>(xa + plane + k);
+                if (M16) xw[u] = *reinterpret_cast<const uint4*>(xb + plane + k);
             }
         }
     };
@@ -198,7 +207,7 @@ smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT*
     // for W.
     constexpr bool AHEAD = !M16 && MODE != SB_ROPE;
     uint4 xn[PER], xwn[PER];
-    if (AHEAD && (int)blockIdx.x < nstrips) load_x(0, xn, xwn);
+    if (AHEAD && (int)blockIdx.x < nstrips) load_x(blockIdx.x, 0, xn, xwn);
     int c = 0;
     for (int strip = blockIdx.x; strip < nstrips; strip += gridDim.x) {
         const int n0 = sb_strip_n0<MODE, NT>(strip, rp);
@@ -216,9 +225,10 @@ smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT*
                     xw[u] = xwn[u];
                 }
                 const bool more = ch + 1 < nch || strip + (int)gridDim.x < nstrips;
-                if (more) load_x(ch + 1 < nch ? ch + 1 : 0, xn, xwn);
+                if (more)
+                    load_x(ch + 1 < nch ? strip : strip + (int)gridDim.x, ch + 1 < nch ? ch + 1 : 0, xn, xwn);
             } else {
-                load_x(ch, xv, xw);
+                load_x(strip, ch, xv, xw);
             }
             // one outcome for the warp: the matrix instructions below are warp-wide
             if (!__all_sync(0xffffffffu, mbar_wait(full + 8 * st, (uint32_t)(c / SB_STAGES) & 1u))) {
@@ -315,7 +325,8 @@ smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT*
                     // act 2: the tanh form of gelu, 0.5 g (1 + tanh z) = g / (1 + exp(-2 z))
                     const float z = rp.act == 2
                         ? 1.5957691216057308f * (gate + 0.044715f * gate * gate * gate) : gate;
-                    y = gate / (1.f + expf(-z)) * up;
+                    y = rp.act == 3 ? clamped_swish(gate, up, rp.limit, rp.alpha)
+                                    : gate / (1.f + expf(-z)) * up;
                 }
                 sb_store<OutT>(out + (size_t)m * ldo + n, y);
             }
@@ -373,10 +384,12 @@ static int pick_nt(int n_out, bool gated, bool m16) {
 
 template <bool GATED, bool M16, typename OutT>
 static int launch_bulk(const bf16* x, const bf16* W, OutT* out, int M, int n_out, int K, int ldx, int ldw,
-                       int ldo, int inter, int w_static, int* error_word, cudaStream_t s, int act = 0) {
-    SbRope rp{};
+                       int ldo, int inter, int w_static, int* error_word, cudaStream_t s, int act = 0,
+                       SbRope rp = SbRope{}) {
     rp.act = act;
-    switch (pick_nt(n_out, GATED, M16)) {
+    int nt = pick_nt(n_out, GATED, M16);
+    while (rp.plane_rows > 0 && nt > 1 && rp.plane_rows % (8 * nt) != 0) nt /= 2;   // a strip has one plane
+    switch (nt) {
         case 4:
             if constexpr (!GATED)
                 return launch_bulk_nt<GATED ? SB_GATED : SB_PLAIN, M16, 4, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
@@ -386,7 +399,8 @@ static int launch_bulk(const bf16* x, const bf16* W, OutT* out, int M, int n_out
 }
 
 // out[M, N] = x W^T (gated == 0), or out[M, N/2] = act(x Wg^T) * (x Wu^T) for W = [Wg; Wu]
-// (gated == 1: act the SiLU, gated == 2: the tanh form of gelu; N even, bfloat16 out).  x: [M, K] bf16 with row stride ldx, W: [N, K] bf16 with
+// (gated == 1: act the SiLU, gated == 2: the tanh form of gelu, gated == 3: the clamped swish with
+// limit and alpha; N even, bfloat16 out).  x: [M, K] bf16 with row stride ldx, W: [N, K] bf16 with
 // row stride ldw, out: bf16 or float (out_dtype) with row stride ldo.  Returns 0, a CUDA error
 // code, or -1 when the shape is refused: M outside 1..16, K no multiple of 32, leading
 // dimensions not multiples of 8 elements or pointers not 16-byte aligned (bulk copies), N odd
@@ -395,7 +409,8 @@ static int launch_bulk(const bf16* x, const bf16* W, OutT* out, int M, int n_out
 // `error_word`: device int, set to 13 / 14 if a bounded wait ran out.
 MSTAR_API int mstar_gemm_smallm_bulk_bf16(const void* x, const void* W, void* out, int M, int N, int K,
                                           int ldx, int ldw, int ldo, int gated, int out_dtype,
-                                          int w_static, int* error_word, void* stream) {
+                                          int w_static, int* error_word, float limit, float alpha,
+                                          void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 16 || K <= 0 || K % 32 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || error_word == nullptr) return -1;
     if (((uintptr_t)x & 15) != 0 || ((uintptr_t)W & 15) != 0) return -1;
@@ -404,10 +419,13 @@ MSTAR_API int mstar_gemm_smallm_bulk_bf16(const void* x, const void* W, void* ou
     const bf16* xp = (const bf16*)x;
     const bf16* wp = (const bf16*)W;
     if (gated) {
-        const int act = gated == 2 ? 2 : 0;
+        const int act = gated >= 2 ? gated : 0;
+        SbRope rp{};
+        rp.limit = limit;
+        rp.alpha = alpha;
         if (M > 8)
-            return launch_bulk<true, true, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act);
-        return launch_bulk<true, false, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act);
+            return launch_bulk<true, true, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act, rp);
+        return launch_bulk<true, false, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act, rp);
     }
     if (out_dtype == MSTAR_F32) {
         if (M > 8) return launch_bulk<false, true, float>(xp, wp, (float*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
@@ -415,6 +433,28 @@ MSTAR_API int mstar_gemm_smallm_bulk_bf16(const void* x, const void* W, void* ou
     }
     if (M > 8) return launch_bulk<false, true, bf16>(xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
     return launch_bulk<false, false, bf16>(xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
+}
+
+// out[M, N] = float products of the rows of W with several planes of x: features [p plane_rows, (p
+// + 1) plane_rows) with x + p plane_stride, the last of `planes` taking the rest.  Refusals as
+// above, and plane_rows and plane_stride multiples of 8.
+MSTAR_API int mstar_gemm_smallm_bulk_planes(const void* x, const void* W, float* out, int M, int N, int K,
+                                            int ldx, int ldw, int ldo, int plane_rows, int planes,
+                                            long long plane_stride, int w_static, int* error_word,
+                                            void* stream) {
+    if (M <= 0 || N <= 0) return 0;
+    if (M > 16 || K <= 0 || K % 32 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || error_word == nullptr) return -1;
+    if (((uintptr_t)x & 15) != 0 || ((uintptr_t)W & 15) != 0) return -1;
+    if (plane_rows <= 0 || plane_rows % 8 != 0 || planes < 1 || plane_stride % 8 != 0) return -1;
+    SbRope rp{};
+    rp.plane_rows = plane_rows;
+    rp.planes = planes;
+    rp.plane_stride = plane_stride;
+    if (M > 8)
+        return launch_bulk<false, true, float>((const bf16*)x, (const bf16*)W, out, M, N, K, ldx, ldw, ldo, 0,
+                                               w_static, error_word, (cudaStream_t)stream, 0, rp);
+    return launch_bulk<false, false, float>((const bf16*)x, (const bf16*)W, out, M, N, K, ldx, ldw, ldo, 0,
+                                            w_static, error_word, (cudaStream_t)stream, 0, rp);
 }
 
 // out[M, N] = relu(x W^T)^2 in bfloat16: the plain product with the activation of a feed-forward

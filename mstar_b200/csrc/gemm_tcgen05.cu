@@ -424,7 +424,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS)
 gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a,
                                const __grid_constant__ CUtensorMap map_b, OutT* __restrict__ out, int M,
                                int N, int K, int ldo, int tiles_m, int tiles_total,
-                               int* __restrict__ error_word, int gate_act) {
+                               int* __restrict__ error_word, int gate_act, float limit, float alpha) {
     static_assert(BN == 256 || BN == 192 || BN == 128, "pair tile width");
     static_assert(!GATED || BN == 256, "the gated form keeps gate and up in 128 columns each");
     constexpr int OUT_COLS = GATED ? BN / 2 : BN;
@@ -594,7 +594,9 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a,
                         // gate_act 1: the tanh form of gelu, 0.5 g (1 + tanh z) = g / (1 + exp(-2 z))
                         const float z = gate_act == 1
                             ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;
-                        r[i] = __float_as_uint(g / (1.f + expf(-z)) * v);
+                        // 2: the clamped swish
+                        r[i] = __float_as_uint(gate_act == 2 ? clamped_swish(g, v, limit, alpha)
+                                                             : g / (1.f + expf(-z)) * v);
                     }
                     const int col = n0 + c0;
                     if (row < M && col < N)
@@ -615,7 +617,8 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a,
 
 template <int BN, int STAGES, bool GATED, typename OutT>
 static int launch_tc_persistent(const CUtensorMap& ma, const CUtensorMap& mb, OutT* out, int M, int N,
-                                int K, int ldo, int* error_word, cudaStream_t s, int gate_act = 0) {
+                                int K, int ldo, int* error_word, cudaStream_t s, int gate_act = 0,
+                                float limit = 0.f, float alpha = 0.f) {
     const size_t smem = (size_t)STAGES * (TC_BM + BN / 2) * TC_BK * 2 + 1024;
     static bool configured = false;
     if (!configured) {
@@ -631,7 +634,7 @@ static int launch_tc_persistent(const CUtensorMap& ma, const CUtensorMap& mb, Ou
     const int on_gpu = pairs_on_gpu();
     const int pairs = total < on_gpu ? total : on_gpu;
     gemm_tcgen05_persistent_kernel<BN, STAGES, GATED, OutT><<<2 * pairs, TC_THREADS, smem, s>>>(
-        ma, mb, out, M, N, K, ldo, tiles_m, total, error_word, gate_act);
+        ma, mb, out, M, N, K, ldo, tiles_m, total, error_word, gate_act, limit, alpha);
     return launch_status();
 }
 
@@ -681,12 +684,13 @@ static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mb, OutT* out, in
 // operands not 16-byte aligned, bn not 128 or 256), -3 / -4 when the tensor map cannot
 // be made.
 // out[M, N/2] = act(x Wg^T) * (x Wu^T) for the fused W = [Wg; Wu] of N rows, bfloat16, on
-// pairs of CTAs; gate_act 0: the SiLU, 1: the tanh form of gelu.  Refusals and error word as
+// pairs of CTAs; gate_act 0: the SiLU, 1: the tanh form of gelu, 2: the clamped swish
+// (limit, alpha).  Refusals and error word as
 // mstar_gemm_tcgen05_bf16; N/2 must be a multiple of 8.
 MSTAR_API int mstar_gemm_tcgen05_gated_bf16(const void* x, const void* W, void* out, int M, int N,
                                             int K, int ldx, int ldw, int ldo, int* error_word,
-                                            int gate_act, void* stream) {
-    if (gate_act != 0 && gate_act != 1) return -1;
+                                            int gate_act, float limit, float alpha, void* stream) {
+    if (gate_act < 0 || gate_act > 2) return -1;
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || N % 16 != 0) return -1;
     if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(W) & 15)) return -1;
@@ -696,7 +700,7 @@ MSTAR_API int mstar_gemm_tcgen05_gated_bf16(const void* x, const void* W, void* 
     rc = make_map(&mb, W, N, K, ldw, 128);
     if (rc != 0) return rc;
     return launch_tc_persistent<256, 6, true, bf16>(ma, mb, (bf16*)out, M, N / 2, K, ldo, error_word,
-                                                    (cudaStream_t)stream, gate_act);
+                                                    (cudaStream_t)stream, gate_act, limit, alpha);
 }
 
 MSTAR_API int mstar_gemm_tcgen05_bf16(const void* x, const void* W, void* out, int M, int N, int K,

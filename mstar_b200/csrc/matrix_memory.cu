@@ -21,8 +21,9 @@
 //
 // State slot layout (floats): S^T [heads][vdim][dim], then n [heads][dim], then m [heads].
 //
-// The second kernel finishes the cell: each head's output is divided by its root mean
-// square, scaled by a weight and gated by sigmoid(g).
+// The second kernel finishes a recurrent mixer: each head's (or equal part's) output is divided
+// by its root mean square, scaled by a weight and gated by sigmoid(g) or silu(g), after the norm or
+// before it.
 #include "common.cuh"
 #include "mma_util.cuh"
 
@@ -284,12 +285,16 @@ MSTAR_API int mstar_matrix_memory_scan(const void* qkv, int act_dtype, int ld, i
     return launch_status();
 }
 
-// out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * weight[h, :] * sigmoid(gate[t, h, :]); one warp
-// per (token, head) where there are many, a block of four warps where there are few; float sums.
-template <typename A, bool BLOCK>
-__global__ void head_norm_gate_kernel(const float* __restrict__ o, const A* __restrict__ gate, int ldg,
+// out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * weight[h, :] * act(gate[t, h, :]), act the
+// sigmoid or (silu 1) the SiLU; with gate_first o act(gate) is normed and scaled.  One warp per
+// (token, head) where there are many, a block of four warps where there are few or the parts
+// are long; float sums.
+__device__ __forceinline__ float hn_gate(float g, int silu) { return (silu ? g : 1.f) / (1.f + expf(-g)); }
+
+template <typename A, typename G, bool BLOCK>
+__global__ void head_norm_gate_kernel(const float* __restrict__ o, const G* __restrict__ gate, int ldg,
                                       const float* __restrict__ weight, A* __restrict__ out,
-                                      int pairs, int heads, int vdim, float eps) {
+                                      int pairs, int heads, int vdim, float eps, int silu, int gate_first) {
     __shared__ float scratch[32];
     const unsigned long long waited = pdl_wait();
     o = pdl_after(o, waited);
@@ -299,33 +304,38 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const A* __re
     const int first = BLOCK ? threadIdx.x : (threadIdx.x & 31), step = BLOCK ? blockDim.x : 32;
     const int t = pair / heads, h = pair - t * heads;
     const float* row = o + (size_t)pair * vdim;
+    const G* g = gate + (size_t)t * ldg + (size_t)h * vdim;
     float ss = 0.f;
-    for (int j = first; j < vdim; j += step) ss = fmaf(row[j], row[j], ss);
+    for (int j = first; j < vdim; j += step) {
+        const float v = gate_first ? row[j] * hn_gate(to_float(g[j]), silu) : row[j];
+        ss = fmaf(v, v, ss);
+    }
     const float total = BLOCK ? block_sum(ss, scratch) : warp_sum(ss);
     const float inv = rsqrtf(total / (float)vdim + eps);
-    const A* g = gate + (size_t)t * ldg + (size_t)h * vdim;
-    for (int j = first; j < vdim; j += step) {
-        const float gv = to_float(g[j]);
-        out[(size_t)pair * vdim + j] =
-            from_float<A>(row[j] * inv * weight[(size_t)h * vdim + j] / (1.f + expf(-gv)));
-    }
+    for (int j = first; j < vdim; j += step)
+        out[(size_t)pair * vdim + j] = from_float<A>(
+            row[j] * inv * weight[(size_t)h * vdim + j] * hn_gate(to_float(g[j]), silu));
 }
 
-MSTAR_API int mstar_head_norm_gate(const float* o, const void* gate, int ldg, const float* weight,
-                                   void* out, int act_dtype, int tokens, int heads, int vdim,
-                                   float eps, void* stream) {
+// `gate_dtype`: the activation type, or float.
+MSTAR_API int mstar_head_norm_gate(const float* o, const void* gate, int gate_dtype, int ldg,
+                                   const float* weight, void* out, int act_dtype, int tokens, int heads,
+                                   int vdim, float eps, int silu, int gate_first, void* stream) {
     if (tokens <= 0) return 0;
+    if (act_dtype == MSTAR_F32 && gate_dtype != MSTAR_F32) return -1;
     cudaStream_t s = (cudaStream_t)stream;
     const int pairs = tokens * heads, warps = 4;
-    const bool few = pairs < 4 * device_sm_count();
+    const bool few = pairs < 4 * device_sm_count() || vdim >= 1024;
     dim3 grid(few ? pairs : (pairs + warps - 1) / warps);
-#define LAUNCH(A, B)                                                                              \
-    mstar_launch((head_norm_gate_kernel<A, B>), grid, dim3(32 * warps), 0, s, o, (const A*)gate, ldg, \
-                 weight, (A*)out, pairs, heads, vdim, eps)
+#define LAUNCH(A, G, B)                                                                           \
+    mstar_launch((head_norm_gate_kernel<A, G, B>), grid, dim3(32 * warps), 0, s, o, (const G*)gate, ldg, \
+                 weight, (A*)out, pairs, heads, vdim, eps, silu, gate_first)
     if (act_dtype == MSTAR_F32) {
-        if (few) LAUNCH(float, true); else LAUNCH(float, false);
+        if (few) LAUNCH(float, float, true); else LAUNCH(float, float, false);
+    } else if (gate_dtype == MSTAR_F32) {
+        if (few) LAUNCH(bf16, float, true); else LAUNCH(bf16, float, false);
     } else {
-        if (few) LAUNCH(bf16, true); else LAUNCH(bf16, false);
+        if (few) LAUNCH(bf16, bf16, true); else LAUNCH(bf16, bf16, false);
     }
 #undef LAUNCH
     return launch_status();

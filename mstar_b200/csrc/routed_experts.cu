@@ -6,8 +6,10 @@
 //           by the sum of the chosen scores when `renormalize`
 //           With a `choice_bias` the largest of s + bias are chosen; the weights stay s.
 //   expert  y = W_down (silu(W_gate u) * (W_up u)),  u = w x (`scale_input`) or u = x with
-//           w multiplying y; without a gate (`gated` 0) y = W_down relu(W_up u)^2
-//   out[t] = sum over the chosen experts (+ `add[t]`, the shared expert's output)
+//           w multiplying y; without a gate (`gated` 0) y = W_down relu(W_up u)^2; `gated` 2
+//           takes the clamped swish of common.cuh (limit, alpha) for the SiLU and the product
+//   out[t] = sum over the chosen experts (+ `add[t]`, the shared expert's output, times
+//           sigmoid(add_gate[t]) where there is such a gate)
 // A chosen index at or beyond `real` (the experts that have matrices) is an identity
 // expert: it adds w x[t].
 //
@@ -30,12 +32,12 @@
 __global__ void route_topk_kernel(const float* __restrict__ logits, const float* __restrict__ choice_bias,
                                   int* __restrict__ chosen,
                                   float* __restrict__ weight, int tokens, int experts, int top,
-                                  int softmax, int renormalize) {
+                                  int softmax, int renormalize, int ld) {
     logits = pdl_after(logits, pdl_wait());
     const int lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (t >= tokens) return;
-    const float* z = logits + (size_t)t * experts;
+    const float* z = logits + (size_t)t * ld;
     float zmax = -INFINITY, denom = 1.f;
     if (softmax) {
         for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, z[e]);
@@ -87,11 +89,12 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, const float*
 
 MSTAR_API int mstar_route_topk(const float* logits, const float* choice_bias, int* chosen,
                                float* weight, int tokens, int experts, int top, int softmax,
-                               int renormalize, void* stream) {
+                               int renormalize, int ld, void* stream) {
     if (tokens <= 0) return 0;
+    if (ld < experts) return -1;
     if (experts <= 0 || top <= 0 || top > experts || experts > 32 * RT_PER_LANE) return -1;
     mstar_launch(route_topk_kernel, dim3((tokens + 3) / 4), dim3(128), 0, (cudaStream_t)stream,
-                 logits, choice_bias, chosen, weight, tokens, experts, top, softmax, renormalize);
+                 logits, choice_bias, chosen, weight, tokens, experts, top, softmax, renormalize, ld);
     return launch_status();
 }
 
@@ -106,7 +109,7 @@ __global__ void __launch_bounds__(RE_THREADS)
 expert_gate_up_kernel(const A* __restrict__ x, const A* __restrict__ w_gate_up,
                       const int* __restrict__ chosen, const float* __restrict__ weight,
                       float* __restrict__ act, int width, int ff, int top, int scale_input,
-                      int real) {
+                      int real, int clamped, float limit, float alpha) {
     extern __shared__ float xs[];            // [width]
     const int row = blockIdx.x, t = row / top;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -161,7 +164,7 @@ expert_gate_up_kernel(const A* __restrict__ x, const A* __restrict__ w_gate_up,
             float v;
             if (GATED) {
                 const float up = warp_sum(su[k]) * w;
-                v = g / (1.f + expf(-g)) * up;
+                v = clamped ? clamped_swish(g, up, limit, alpha) : g / (1.f + expf(-g)) * up;
             } else {
                 const float r = fmaxf(g, 0.f);
                 v = r * r;
@@ -177,7 +180,8 @@ __global__ void __launch_bounds__(RE_THREADS)
 expert_down_kernel(const float* __restrict__ act, const A* __restrict__ w_down,
                    const int* __restrict__ chosen, const float* __restrict__ weight,
                    const A* __restrict__ add, A* __restrict__ out, int width, int ff, int top,
-                   int scale_input, const A* __restrict__ x, int real) {
+                   int scale_input, const A* __restrict__ x, int real, const float* add_gate,
+                   int gate_stride) {
     extern __shared__ float as[];            // [top][ff]
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -185,6 +189,8 @@ expert_down_kernel(const float* __restrict__ act, const A* __restrict__ w_down,
     act = pdl_after(act, waited);
     add = pdl_after(add, waited);
     x = pdl_after(x, waited);
+    add_gate = pdl_after(add_gate, waited);
+    const float share = add_gate == nullptr ? 1.f : 1.f / (1.f + expf(-add_gate[(size_t)t * gate_stride]));
     for (int i = threadIdx.x; i < top * ff; i += RE_THREADS)
         as[i] = chosen[(size_t)t * top + i / ff] < real ? act[(size_t)t * top * ff + i] : 0.f;
     __syncthreads();
@@ -233,7 +239,7 @@ expert_down_kernel(const float* __restrict__ act, const A* __restrict__ w_down,
                 const int c = c0 + q;
                 if (c < c_end) {
                     float v = total[q];
-                    if (add != nullptr) v += to_float(add[(size_t)t * width + c]);
+                    if (add != nullptr) v += share * to_float(add[(size_t)t * width + c]);
                     out[(size_t)t * width + c] = from_float<A>(v);
                 }
             }
@@ -248,7 +254,8 @@ MSTAR_API int mstar_experts_by_row(const void* x, const void* w_gate_up, const v
                                    const int* chosen, const float* weight, float* act,
                                    const void* add, void* out, int act_dtype, int tokens,
                                    int width, int ff, int top, int scale_input, int gated,
-                                   int real, void* stream) {
+                                   int real, float limit, float alpha, const float* add_gate,
+                                   int gate_stride, void* stream) {
     if (tokens <= 0) return 0;
     if (width <= 0 || ff <= 0 || top <= 0) return -1;
     if ((size_t)width * 4 > 48 * 1024 || (size_t)top * ff * 4 > 48 * 1024) return -1;
@@ -257,17 +264,17 @@ MSTAR_API int mstar_experts_by_row(const void* x, const void* w_gate_up, const v
 #define GO(A, GATED)                                                                              \
     mstar_launch((expert_gate_up_kernel<A, GATED>), g1, dim3(RE_THREADS), sizeof(float) * width, s, \
                  (const A*)x, (const A*)w_gate_up, chosen, weight, act, width, ff, top,            \
-                 scale_input, real)
+                 scale_input, real, (int)(gated == 2), limit, alpha)
     if (act_dtype == MSTAR_F32) {
         if (gated) { GO(float, true); } else { GO(float, false); }
         mstar_launch((expert_down_kernel<float>), g2, dim3(RE_THREADS), sizeof(float) * top * ff, s,
                      (const float*)act, (const float*)w_down, chosen, weight, (const float*)add,
-                     (float*)out, width, ff, top, scale_input, (const float*)x, real);
+                     (float*)out, width, ff, top, scale_input, (const float*)x, real, add_gate, gate_stride);
     } else {
         if (gated) { GO(bf16, true); } else { GO(bf16, false); }
         mstar_launch((expert_down_kernel<bf16>), g2, dim3(RE_THREADS), sizeof(float) * top * ff, s,
                      (const float*)act, (const bf16*)w_down, chosen, weight, (const bf16*)add,
-                     (bf16*)out, width, ff, top, scale_input, (const bf16*)x, real);
+                     (bf16*)out, width, ff, top, scale_input, (const bf16*)x, real, add_gate, gate_stride);
     }
 #undef GO
     return launch_status();
@@ -339,7 +346,7 @@ grouped_gemm_kernel(const bf16* __restrict__ a_src, const bf16* __restrict__ w, 
                     const int* __restrict__ order, const float* __restrict__ weight,
                     const int* __restrict__ offsets, const int* __restrict__ tile_expert,
                     const int* __restrict__ tile_first, const int* __restrict__ num_tiles,
-                    int N, int K, int top, int scale_input) {
+                    int N, int K, int top, int scale_input, int clamped, float limit, float alpha) {
     constexpr bool GATED = MODE == 1;
     constexpr bool GATHER = MODE != 0;
     constexpr int BROWS = GATED ? 2 * GG_BN : GG_BN;
@@ -454,8 +461,11 @@ grouped_gemm_kernel(const bf16* __restrict__ a_src, const bf16* __restrict__ w, 
                     const float u0 = acc[GATED ? 1 : 0][i][j][half * 2] * wgt;
                     const float u1 = acc[GATED ? 1 : 0][i][j][half * 2 + 1] * wgt;
                     bf16* o = (bf16*)out + (size_t)p * N + n;
-                    o[0] = __float2bfloat16_rn(g0 / (1.f + expf(-g0)) * u0);
-                    if (n + 1 < N) o[1] = __float2bfloat16_rn(g1 / (1.f + expf(-g1)) * u1);
+                    o[0] = __float2bfloat16_rn(clamped ? clamped_swish(g0, u0, limit, alpha)
+                                                       : g0 / (1.f + expf(-g0)) * u0);
+                    if (n + 1 < N)
+                        o[1] = __float2bfloat16_rn(clamped ? clamped_swish(g1, u1, limit, alpha)
+                                                           : g1 / (1.f + expf(-g1)) * u1);
                 } else if (MODE == 2) {
                     const float r0 = fmaxf(acc[0][i][j][half * 2] * wgt, 0.f);
                     const float r1 = fmaxf(acc[0][i][j][half * 2 + 1] * wgt, 0.f);
@@ -477,12 +487,14 @@ __global__ void experts_combine_kernel(const float* __restrict__ y, const int* _
                                        const float* __restrict__ weight, const A* __restrict__ add,
                                        A* __restrict__ out, int width, int top, int scale_input,
                                        const int* __restrict__ chosen, const A* __restrict__ x,
-                                       int real) {
+                                       int real, const float* add_gate, int gate_stride) {
     const unsigned long long waited = pdl_wait();
     y = pdl_after(y, waited);
     pos = pdl_after(pos, waited);
     add = pdl_after(add, waited);
+    add_gate = pdl_after(add_gate, waited);
     const int t = blockIdx.x;
+    const float share = add_gate == nullptr ? 1.f : 1.f / (1.f + expf(-add_gate[(size_t)t * gate_stride]));
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float total = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -493,7 +505,7 @@ __global__ void experts_combine_kernel(const float* __restrict__ y, const int* _
             const float v = y[(size_t)pos[(size_t)t * top + k] * width + c];
             total += scale_input ? v : v * weight[(size_t)t * top + k];
         }
-        if (add != nullptr) total += to_float(add[(size_t)t * width + c]);
+        if (add != nullptr) total += share * to_float(add[(size_t)t * width + c]);
         out[(size_t)t * width + c] = from_float<A>(total);
     }
 }
@@ -505,7 +517,8 @@ MSTAR_API int mstar_experts_grouped(const void* x, const void* w_gate_up, const 
                                     const int* chosen, const float* weight, int* ints, void* act,
                                     float* y, const void* add, void* out, int tokens, int width,
                                     int ff, int top, int experts, int scale_input, int gated,
-                                    int real, void* stream) {
+                                    int real, float limit, float alpha, const float* add_gate,
+                                    int gate_stride, void* stream) {
     if (tokens <= 0) return 0;
     if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 1024 || top <= 0) return -1;
     cudaStream_t s = (cudaStream_t)stream;
@@ -538,24 +551,24 @@ MSTAR_API int mstar_experts_grouped(const void* x, const void* w_gate_up, const 
 #define GG_UP(BM)                                                                                 \
     if (gated)                                                                                    \
         GG_GO(1, BM, 2 * GG_BN, gx1, (const bf16*)x, (const bf16*)w_gate_up, act, order, weight,  \
-              offsets, tile_expert, tile_first, num_tiles, ff, width, top, scale_input)           \
+              offsets, tile_expert, tile_first, num_tiles, ff, width, top, scale_input, (int)(gated == 2), limit, alpha)           \
     else                                                                                          \
         GG_GO(2, BM, GG_BN, gx1, (const bf16*)x, (const bf16*)w_gate_up, act, order, weight,      \
-              offsets, tile_expert, tile_first, num_tiles, ff, width, top, scale_input)
+              offsets, tile_expert, tile_first, num_tiles, ff, width, top, scale_input, (int)(gated == 2), limit, alpha)
     if (bm == 128) {
         GG_UP(128)
         GG_GO(0, 128, GG_BN, gx2, (const bf16*)act, (const bf16*)w_down, (void*)y, order, weight,
-              offsets, tile_expert, tile_first, num_tiles, width, ff, top, scale_input)
+              offsets, tile_expert, tile_first, num_tiles, width, ff, top, scale_input, 0, 0.f, 0.f)
     } else {
         GG_UP(64)
         GG_GO(0, 64, GG_BN, gx2, (const bf16*)act, (const bf16*)w_down, (void*)y, order, weight,
-              offsets, tile_expert, tile_first, num_tiles, width, ff, top, scale_input)
+              offsets, tile_expert, tile_first, num_tiles, width, ff, top, scale_input, 0, 0.f, 0.f)
     }
 #undef GG_UP
 #undef GG_GO
 #undef GG_SMEM
     mstar_launch((experts_combine_kernel<bf16>), dim3(tokens), dim3(256), 0, s, (const float*)y, pos,
                  weight, (const bf16*)add, (bf16*)out, width, top, scale_input, chosen,
-                 (const bf16*)x, real);
+                 (const bf16*)x, real, add_gate, gate_stride);
     return launch_status();
 }

@@ -39,6 +39,10 @@ def model_param_specs(layout: ModelLayout) -> dict:
     norm_cls = part_class("norm", layout.final_norm)
     for local, ps in norm_cls.param_specs(layout.final_norm).items():
         specs[f"final_norm.{local}"] = ps
+    if layout.loop_input is not None:
+        cls = part_class("loop_input", layout.loop_input)
+        for local, ps in cls.param_specs(layout.loop_input).items():
+            specs[f"loop_input.{local}"] = ps
     head = layout.head_spec()
     for local, ps in part_class("head", head).param_specs(head).items():
         specs[f"head.{local}"] = ps
@@ -77,12 +81,19 @@ class Model:
                        for i, spec in enumerate(layout.blocks)]
         self.final_norm = build_part("norm", layout.final_norm, _sub(params, "final_norm"),
                                      runtime)
+        self.loop_input = None
+        if layout.loop_input is not None:
+            self.loop_input = build_part("loop_input", layout.loop_input,
+                                         _sub(params, "loop_input"), runtime)
+            # blocks that add into the residual tensor itself get one of their own each pass
+            self.loop_input.shared = all(getattr(b, "keeps_residual", False) for b in self.blocks)
         self.cache_needs = cache_needs(layout)
         # a decode step may be captured as a CUDA graph only if every block says that its
         # forward pass reads nothing per-step from the host; a block that says nothing is
         # taken as unsafe
         self.graph_safe = all(getattr(p, "graph_safe", False) is True
-                              for p in (self.embedding, self.head, self.final_norm, *self.blocks))
+                              for p in (self.embedding, self.head, self.final_norm, *self.blocks,
+                                        *([self.loop_input] if self.loop_input else [])))
 
     @property
     def vocab_size(self) -> int:
@@ -106,7 +117,10 @@ class Model:
                 want_rows: Optional[torch.Tensor]) -> torch.Tensor:
         """Run the tokens of one step; return float logits [len(want_rows), vocab]."""
         stream = ResidualStream(self.embedding.forward(token_ids, ctx))
+        anchor = self.loop_input.begin(stream.h) if self.loop_input is not None else None
         for entry in self.layout.order:
+            if entry.loop_input:
+                self.loop_input.apply(stream, anchor)
             self.blocks[entry.block].forward(stream, ctx, storage.layer_cache(entry.cache,
                                                                                block_tables))
         if want_rows is None or want_rows.numel() == 0:

@@ -112,22 +112,26 @@ def gather_add_rows(resid: torch.Tensor, delta, rows: torch.Tensor):
 
 
 GATE_ACTIVATIONS = {"gelu_tanh": 1, "silu": 2}
+# gated activations that are more than a factor: (limit, alpha) go with them
+GATED_PRODUCTS = {**GATE_ACTIVATIONS, "clamped_swish": 3}
 
 
-def silu_mul(gate_up: torch.Tensor, out=None, kind: str = "silu"):
+def silu_mul(gate_up: torch.Tensor, out=None, kind: str = "silu", limit: float = 0.0,
+             alpha: float = 0.0):
     """act(gate_up[:, :I]) * gate_up[:, I:], act the SiLU or (``kind`` "gelu_tanh") the tanh
-    form of gelu."""
+    form of gelu; "clamped_swish": with g = min(gate, limit) and u = clamp(up, -limit, limit),
+    g * sigmoid(alpha * g) * (u + 1)."""
     _need_cuda(gate_up)
-    if kind not in GATE_ACTIVATIONS:
+    if kind not in GATED_PRODUCTS:
         raise KernelError(f"gate activation {kind!r} has no kernel (known: "
-                          f"{sorted(GATE_ACTIVATIONS)})")
+                          f"{sorted(GATED_PRODUCTS)})")
     assert gate_up.dim() == 2 and gate_up.is_contiguous() and gate_up.shape[1] % 2 == 0
     rows, inter = gate_up.shape[0], gate_up.shape[1] // 2
     if out is None:
         out = torch.empty((rows, inter), dtype=gate_up.dtype, device=gate_up.device)
     check(lib.get("elementwise").mstar_silu_mul(
-        gate_up.data_ptr(), out.data_ptr(), _dt(gate_up), rows, inter, GATE_ACTIVATIONS[kind],
-        _stream()), "silu_mul")
+        gate_up.data_ptr(), out.data_ptr(), _dt(gate_up), rows, inter, GATED_PRODUCTS[kind],
+        float(limit), float(alpha), _stream()), "silu_mul")
     return out
 
 
@@ -414,20 +418,48 @@ def _smallm_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def _gemm_smallm(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, gated,
-                 static_weights: bool = False):
+                 static_weights: bool = False, limit: float = 0.0, alpha: float = 0.0):
     """``gated``: False or 0 for the plain product; True or 1 gates by the SiLU, 2 by the tanh
-    form of gelu."""
+    form of gelu, 3 by the clamped swish with ``limit`` and ``alpha``."""
     m, k = x.shape
     n = w.shape[0]
     out = torch.empty((m, n // 2 if gated else n), dtype=out_dtype, device=x.device)
     code = lib.get("gemm_smallm_bulk").mstar_gemm_smallm_bulk_bf16(
         x.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, x.stride(0), w.stride(0),
         out.stride(0), int(gated), _dt(out), int(static_weights),
-        tcgen05_error_word(x.device).data_ptr(), _stream())
+        tcgen05_error_word(x.device).data_ptr(), float(limit), float(alpha), _stream())
     if code == -1:
         raise KernelError(f"small-M GEMM refuses M={m}, N={n}, K={k}")
     check(code, "gemm_smallm_bulk")
     return out
+
+
+def linear_planes(x: torch.Tensor, w: torch.Tensor, plane_rows: int,
+                  static_weights: bool = False) -> tuple:
+    """Products of row groups of ``w`` [N, K] with inputs of their own: rows [p * plane_rows, (p +
+    1) * plane_rows) of w meet plane p of ``x`` [planes, M, K], the last plane takes the rows that
+    are left.  Returns float (the products of the planes before the last side by side, [M,
+    (planes - 1) * plane_rows], the last plane's).  One weight-streaming kernel for few bfloat16
+    rows (MSTAR_PLANES=0: never); else a batched product and one for the last plane."""
+    _need_cuda(x, w)
+    assert x.dim() == 3 and x.is_contiguous() and w.is_contiguous() and w.shape[1] == x.shape[2]
+    planes, m, k = x.shape
+    n, full = w.shape[0], planes - 1
+    assert planes > 1 and n > full * plane_rows
+    if _smallm_ok(x[0], w) and plane_rows % 8 == 0 and os.environ.get("MSTAR_PLANES") != "0":
+        out = torch.empty((m, n), dtype=torch.float32, device=x.device)
+        code = lib.get("gemm_smallm_bulk").mstar_gemm_smallm_bulk_planes(
+            x.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, k, k, n, plane_rows, planes, m * k,
+            int(static_weights), tcgen05_error_word(x.device).data_ptr(), _stream())
+        if code == -1:
+            raise KernelError(f"small-M GEMM refuses M={m}, N={n}, K={k}, planes of {plane_rows} rows")
+        check(code, "gemm_smallm_bulk_planes")
+        return out[:, :full * plane_rows], out[:, full * plane_rows:]
+    head = linear_per_head(x[:full].transpose(0, 1), w[:full * plane_rows].view(full, plane_rows, k),
+                           out_dtype=torch.float32).view(m, full * plane_rows)
+    tail = linear(x[full], w[full * plane_rows:], out_dtype=torch.float32,
+                  static_weights=static_weights)
+    return head, tail
 
 
 # Rows up to which the swapped-operand tcgen05 kernel is used (tokens are the MMA's N
@@ -584,11 +616,13 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None
     return out
 
 
-def gemm_tcgen05_gated(x: torch.Tensor, w_gate_up: torch.Tensor, kind: str = "silu"):
+def gemm_tcgen05_gated(x: torch.Tensor, w_gate_up: torch.Tensor, kind: str = "silu",
+                       limit: float = 0.0, alpha: float = 0.0):
     """act(x Wg^T) * (x Wu^T) for the fused [Wg; Wu] on pairs of CTAs (cta_group::2), the
-    activation (``kind``: "silu" or "gelu_tanh") applied in the epilogue straight from tensor
-    memory."""
-    assert kind in ("silu", "gelu_tanh")
+    activation (``kind``: "silu", "gelu_tanh" or "clamped_swish" with ``limit`` and ``alpha``)
+    applied in the epilogue straight from tensor memory."""
+    code_of = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
+    assert kind in code_of
     _need_cuda(x, w_gate_up)
     assert x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16
     assert x.stride(1) == 1 and w_gate_up.stride(1) == 1 and x.shape[1] == w_gate_up.shape[1]
@@ -598,7 +632,7 @@ def gemm_tcgen05_gated(x: torch.Tensor, w_gate_up: torch.Tensor, kind: str = "si
     code = lib.get("gemm_tcgen05").mstar_gemm_tcgen05_gated_bf16(
         x.data_ptr(), w_gate_up.data_ptr(), out.data_ptr(), m, n, k, x.stride(0),
         w_gate_up.stride(0), out.stride(0), tcgen05_error_word(x.device).data_ptr(),
-        0 if kind == "silu" else 1, _stream())
+        code_of[kind], float(limit), float(alpha), _stream())
     if code == -1:
         raise KernelError(f"gated tcgen05 GEMM refuses M={m}, N={n}, K={k}")
     if code in (-3, -4):
@@ -694,20 +728,22 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, kind: str, static_weights: bool
 
 
 def gated_up(x: torch.Tensor, w_gate_up: torch.Tensor, static_weights: bool = False,
-             kind: str = "silu"):
+             kind: str = "silu", limit: float = 0.0, alpha: float = 0.0):
     """act(x Wg^T) * (x Wu^T) for the fused matrix [Wg; Wu], act the SiLU or (``kind``
-    "gelu_tanh") the tanh form of gelu: one kernel for bfloat16 rows whose shapes the small-M
-    or the tcgen05 kernel takes (MSTAR_FUSED_ACT=0: never for the gelu), else the product
+    "gelu_tanh") the tanh form of gelu ("clamped_swish": see ``silu_mul``): one kernel for bfloat16 rows whose shapes the small-M
+    or the tcgen05 kernel takes (MSTAR_FUSED_ACT=0: only for the SiLU), else the product
     followed by the activation-multiply kernel."""
     _need_cuda(x, w_gate_up)
-    if kind == "silu" or (kind == "gelu_tanh" and os.environ.get("MSTAR_FUSED_ACT") != "0"):
+    if kind == "silu" or (kind in GATED_PRODUCTS and os.environ.get("MSTAR_FUSED_ACT") != "0"):
         if _smallm_ok(x, w_gate_up) and w_gate_up.shape[0] % 2 == 0:
-            return _gemm_smallm(x, w_gate_up, torch.bfloat16, gated=1 if kind == "silu" else 2,
-                                static_weights=static_weights)
+            return _gemm_smallm(x, w_gate_up, torch.bfloat16,
+                                gated={"silu": 1, "gelu_tanh": 2, "clamped_swish": 3}[kind],
+                                static_weights=static_weights, limit=limit, alpha=alpha)
         if (_tc_ok(x, w_gate_up) and w_gate_up.shape[0] % 16 == 0
                 and tcgen05_tile(x.shape[0], w_gate_up.shape[0]) is not None):
-            return gemm_tcgen05_gated(x, w_gate_up, kind)
-    return silu_mul(linear(x, w_gate_up, static_weights=static_weights), kind=kind)
+            return gemm_tcgen05_gated(x, w_gate_up, kind, limit, alpha)
+    return silu_mul(linear(x, w_gate_up, static_weights=static_weights), kind=kind, limit=limit,
+                    alpha=alpha)
 
 
 _argmax_scratch: dict = {}
@@ -940,16 +976,20 @@ def matrix_memory_scan(proj: torch.Tensor, gates: torch.Tensor, bias: torch.Tens
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, heads: int,
-                   vdim: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
-    """o / rms(o per head) * weight * sigmoid(gate): float ``o`` [tokens, heads*vdim], ``gate``
-    a column view in ``out_dtype``, float ``weight`` [heads*vdim]."""
+                   vdim: int, eps: float, out_dtype: torch.dtype, kind: str = "sigmoid",
+                   gate_first: bool = False) -> torch.Tensor:
+    """o / rms(o per head) * weight * act(gate): float ``o`` [tokens, heads*vdim], ``gate`` a
+    column view in ``out_dtype`` or float, float ``weight`` [heads*vdim]; act (``kind``) the
+    "sigmoid" or the "silu".  ``gate_first``: o * act(gate) is what is normed and scaled."""
     _need_cuda(o, gate, weight)
+    assert kind in ("sigmoid", "silu")
     assert o.dtype == torch.float32 and o.is_contiguous() and weight.dtype == torch.float32
-    assert gate.dtype == out_dtype and gate.stride(1) == 1 and gate.shape == o.shape
+    assert gate.dtype in (out_dtype, torch.float32) and gate.stride(1) == 1 and gate.shape == o.shape
     out = torch.empty(o.shape, dtype=out_dtype, device=o.device)
     check(lib.get("matrix_memory").mstar_head_norm_gate(
-        o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), out.data_ptr(), _dt(out),
-        o.shape[0], heads, vdim, float(eps), _stream()), "head_norm_gate")
+        o.data_ptr(), gate.data_ptr(), _dt(gate), gate.stride(0), weight.data_ptr(), out.data_ptr(),
+        _dt(out), o.shape[0], heads, vdim, float(eps), int(kind == "silu"), int(gate_first),
+        _stream()), "head_norm_gate")
     return out
 
 
@@ -1111,10 +1151,11 @@ def linear_per_head(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | N
 # ------------------------------------------------------------------ routed experts
 def route_topk(logits: torch.Tensor, top: int, softmax: bool = False, renormalize: bool = False,
                choice_bias=None):
-    """(chosen int32 [tokens, top], weight float [tokens, top]) from float router logits.
+    """(chosen int32 [tokens, top], weight float [tokens, top]) from float router logits (a
+    column view of a wider product will do).
     ``choice_bias``: float [experts] added to the scores for the choice only."""
     _need_cuda(logits, choice_bias)
-    assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.is_contiguous()
+    assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.stride(1) == 1
     tokens, experts = logits.shape
     assert choice_bias is None or (choice_bias.dtype == torch.float32
                                    and choice_bias.numel() == experts)
@@ -1122,7 +1163,7 @@ def route_topk(logits: torch.Tensor, top: int, softmax: bool = False, renormaliz
     weight = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     code = lib.get("routed_experts").mstar_route_topk(
         logits.data_ptr(), _ptr(choice_bias), chosen.data_ptr(), weight.data_ptr(), tokens, experts, top,
-        int(softmax), int(renormalize), _stream())
+        int(softmax), int(renormalize), logits.stride(0), _stream())
     if code == -1:
         raise KernelError(f"cannot choose {top} of {experts} experts")
     check(code, "route_topk")
@@ -1131,12 +1172,15 @@ def route_topk(logits: torch.Tensor, top: int, softmax: bool = False, renormaliz
 
 def experts_by_row(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, chosen, weight,
                    ff: int, scale_input: bool, add=None, gated: bool = True,
-                   real: int | None = None) -> torch.Tensor:
+                   real: int | None = None, clamp=None, add_gate=None) -> torch.Tensor:
     """sum over a token's chosen experts of down(silu(gate u) * up u) (+ ``add``), every row
     streaming its experts' matrices.  ``w_gate_up``: [experts * 2 * ff, width] (per expert
     gate rows, then up rows), ``w_down``: [experts * width, ff].  ``gated`` False: an expert
     is down(relu(up u)^2) and ``w_gate_up`` [experts * ff, width].  ``real``: experts that
-    have matrices; a chosen index at or beyond it adds weight * x (default: all are real)."""
+    have matrices; a chosen index at or beyond it adds weight * x (default: all are real).
+    ``clamp``: (limit, alpha) makes the gated form the clamped swish (``silu_mul``).
+    ``add_gate``: float [tokens, 1], a column view of a wider product; ``add`` is multiplied by
+    its sigmoid."""
     if real is None:
         real = w_down.shape[0] // x.shape[1]
     _need_cuda(x, w_gate_up, w_down, chosen, weight, add)
@@ -1151,13 +1195,29 @@ def experts_by_row(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tenso
     code = lib.get("routed_experts").mstar_experts_by_row(
         x.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), chosen.data_ptr(),
         weight.data_ptr(), act.data_ptr(), _ptr(add), out.data_ptr(), _dt(x), tokens, width, ff,
-        top, int(scale_input), int(gated), int(real), _stream())
+        top, int(scale_input), _gated_code(gated, clamp), int(real), *(clamp or (0.0, 0.0)),
+        *_add_gate(add_gate, tokens), _stream())
     if code == -1:
         raise KernelError(f"the by-row expert kernels refuse width={width}, ff={ff}, top={top} "
                           "(a row of inputs, and of hidden units, within 48 KB)")
     check(code, "experts_by_row")
     lib.add_launches(1)                       # two kernels behind one call
     return out
+
+
+def _gated_code(gated: bool, clamp) -> int:
+    if clamp is not None and not gated:
+        raise KernelError("the clamped swish is a gated activation")
+    return 2 if clamp is not None else int(gated)
+
+
+def _add_gate(gate, tokens: int) -> tuple:
+    """(pointer, floats between tokens) of a gate column, or nulls."""
+    if gate is None:
+        return 0, 0
+    _need_cuda(gate)
+    assert gate.dtype == torch.float32 and tuple(gate.shape) == (tokens, 1)
+    return gate.data_ptr(), gate.stride(0)
 
 
 # Rows (tokens x choices) from which on the experts' rows are sorted by expert and run as
@@ -1167,7 +1227,7 @@ GROUPED_EXPERT_ROWS = 64
 
 def experts_grouped(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, chosen, weight,
                     experts: int, ff: int, scale_input: bool, add=None, gated: bool = True,
-                    real: int | None = None) -> torch.Tensor:
+                    real: int | None = None, clamp=None, add_gate=None) -> torch.Tensor:
     """The same sums as ``experts_by_row`` for many bfloat16 rows: rows sorted by expert on
     the device, each expert's rows through its matrices as 64-row tiles on the tensor cores
     (float sums), a token's choices added up in their order.  Nothing is read by the host."""
@@ -1190,7 +1250,8 @@ def experts_grouped(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tens
     code = lib.get("routed_experts").mstar_experts_grouped(
         x.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), chosen.data_ptr(),
         weight.data_ptr(), ints.data_ptr(), act.data_ptr(), y.data_ptr(), _ptr(add),
-        out.data_ptr(), tokens, width, ff, top, experts, int(scale_input), int(gated), int(real),
+        out.data_ptr(), tokens, width, ff, top, experts, int(scale_input),
+        _gated_code(gated, clamp), int(real), *(clamp or (0.0, 0.0)), *_add_gate(add_gate, tokens),
         _stream())
     if code == -1:
         raise KernelError(f"the grouped expert kernels refuse width={width}, ff={ff}, "
@@ -1202,7 +1263,7 @@ def experts_grouped(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tens
 
 def routed_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, chosen, weight,
                    experts: int, ff: int, scale_input: bool, add=None, gated: bool = True,
-                   identity: int = 0) -> torch.Tensor:
+                   identity: int = 0, clamp=None, add_gate=None) -> torch.Tensor:
     """sum over a token's chosen experts of down(silu(gate u) * up u) (+ ``add``): sorted by
     expert on the tensor cores from ``GROUPED_EXPERT_ROWS`` bfloat16 rows on
     (MSTAR_EXPERTS=by_row: never), row by row below and in float32."""
@@ -1210,9 +1271,10 @@ def routed_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tenso
     if (x.dtype == torch.bfloat16 and rows >= GROUPED_EXPERT_ROWS and x.shape[1] % 8 == 0
             and ff % 8 == 0 and experts <= 1024 and os.environ.get("MSTAR_EXPERTS") != "by_row"):
         return experts_grouped(x, w_gate_up, w_down, chosen, weight, experts + identity, ff,
-                               scale_input, add, gated=gated, real=experts)
+                               scale_input, add, gated=gated, real=experts, clamp=clamp,
+                               add_gate=add_gate)
     return experts_by_row(x, w_gate_up, w_down, chosen, weight, ff, scale_input, add, gated=gated,
-                          real=experts)
+                          real=experts, clamp=clamp, add_gate=add_gate)
 
 
 # ------------------------------------------------------------------ window attention with kept first keys
@@ -1337,7 +1399,8 @@ def sink_attention_splits(entries: int, max_q_len: int, num_heads: int, num_kv_h
 def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_req, cache_pos,
                    num_heads: int, num_kv_heads: int, head_dim: int, v_dim: int, page_size: int,
                    window: int, keep_first: int, scale: float, ctx=None, gate=None,
-                   softcap: float | None = None, sink=None) -> torch.Tensor:
+                   softcap: float | None = None, sink=None, chunk: int = 0,
+                   sigmoid: bool = False, bias=None) -> torch.Tensor:
     """Softmax attention of every token over the keys it sees: those of the last ``window``
     positions (0: all) and the first ``keep_first`` of the sequence.  ``q``: [tokens, heads *
     head_dim]; returns [tokens, heads * v_dim].  ``gate``: None, or float [tokens, heads] (a
@@ -1345,7 +1408,10 @@ def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_r
     where the tensor-core kernel writes it out, by a kernel of its own after the other; a gate
     of [tokens, heads * v_dim] numbers multiplies feature by feature.  ``softcap``: a score
     becomes ``softcap * tanh(score / softcap)`` after the scale.  ``sink``: float [heads];
-    ``exp(sink[h])`` joins the denominator of head h's softmax (no key, no value).  bfloat16 with sizes that are multiples of 8
+    ``exp(sink[h])`` joins the denominator of head h's softmax (no key, no value).  ``chunk``
+    (instead of a window): a token at position p sees keys from ``p // chunk * chunk`` on.
+    ``bias``: float [heads], added to the capped scores.  ``sigmoid``: the weight of a visible
+    key is the sigmoid of its score, nothing is normalised.  bfloat16 with sizes that are multiples of 8
     up to 256 and a step context (``ctx``: entries, their token ranges and lengths) runs on
     the tensor cores (MSTAR_SINK_ATTENTION=generic: never); everything else, float32
     included, on the CUDA cores."""
@@ -1360,6 +1426,10 @@ def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_r
     if sink is not None:
         _need_cuda(sink)
         assert sink.dtype == torch.float32 and sink.numel() == num_heads and sink.is_contiguous()
+    if bias is not None:
+        _need_cuda(bias)
+        assert bias.dtype == torch.float32 and bias.numel() == num_heads and bias.is_contiguous()
+    assert not (sigmoid and sink is not None) and not (chunk and window)
     cap = float(softcap or 0.0)
     out = torch.empty((tokens, num_heads * v_dim), dtype=q.dtype, device=q.device)
     if (ctx is not None and q.dtype == torch.bfloat16 and head_dim % 8 == 0 and v_dim % 8 == 0
@@ -1367,6 +1437,8 @@ def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_r
         max_keys = ctx.max_kv_len
         if window:
             max_keys = min(max_keys, window + keep_first + ctx.max_q_len)
+        if chunk:
+            max_keys = min(max_keys, chunk + ctx.max_q_len)
         splits = sink_attention_splits(ctx.num_entries, ctx.max_q_len, num_heads, num_kv_heads,
                                        max_keys, num_sms(q.device), wide=max(head_dim, v_dim))
         scratch = None
@@ -1379,7 +1451,7 @@ def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_r
             ctx.num_entries, tokens, ctx.max_q_len, num_heads, num_kv_heads, head_dim, v_dim,
             page_size, int(window or 0), int(keep_first), float(scale), splits, _ptr(scratch),
             _ptr(gate), gate.stride(0) if gate is not None else 0, int(gate_features), cap,
-            _ptr(sink), _stream())
+            _ptr(sink), int(chunk), int(sigmoid), _ptr(bias), _stream())
         if code == -1:
             raise KernelError(f"tensor-core window attention refuses heads={num_heads}, "
                               f"kv_heads={num_kv_heads}, head_dim={head_dim}, v_dim={v_dim}")
@@ -1392,7 +1464,7 @@ def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_r
         block_table.stride(0), token_req.data_ptr(), cache_pos.data_ptr(), tokens, num_heads,
         num_kv_heads, head_dim, v_dim, page_size, int(window or 0), int(keep_first), float(scale),
         _dt(q), cap, _ptr(sink), _ptr(gate) if gate_features else 0,
-        gate.stride(0) if gate_features else 0, _stream())
+        gate.stride(0) if gate_features else 0, int(chunk), int(sigmoid), _ptr(bias), _stream())
     if code == -1:
         raise KernelError(f"window attention refuses heads={num_heads}, kv_heads={num_kv_heads}, "
                           f"head_dim={head_dim}, v_dim={v_dim}")
@@ -1696,4 +1768,266 @@ def delta_finish(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, head
         o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), out.data_ptr(),
         _DT[out_dtype], o.shape[0], heads, vdim, float(eps), float(scale), _stream()),
         "delta_finish")
+    return out
+
+
+# ------------------------------------------------------------------ sublayers side by side
+class SideBySideOutput:
+    """A layer's ``mixer output + feed-forward output``, not added yet: ``mixer`` is a tensor or a
+    ``MeanOfNorms`` of two branches, ``ffn`` a tensor or None.  ``side_step`` adds it to the
+    residual in the kernel that norms it for the next layer."""
+
+    def __init__(self, mixer, ffn=None):
+        if hasattr(mixer, "materialize") and not (isinstance(mixer, MeanOfNorms)
+                                                  and len(mixer.branches) == 2):
+            mixer = mixer.materialize()
+        self.mixer, self.ffn = mixer, ffn
+        self.shape = mixer.shape
+
+    def materialize(self) -> torch.Tensor:
+        y = self.mixer.materialize() if hasattr(self.mixer, "materialize") else self.mixer
+        return y if self.ffn is None else y.float() + self.ffn.float()
+
+    def gather(self, resid: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
+        """float rows of ``resid`` plus this output."""
+        return side_step(resid, self, rows=rows)
+
+
+def side_step(resid: torch.Tensor, pending=None, *, act_dtype=None, rows=None, norm_weight=None,
+              eps: float = 0.0, normed: bool = False, shift=None, prev=None, ctx=None,
+              raw: bool = False):
+    """The step between two layers with sublayers side by side: x = ``resid`` (float, left as
+    it is) + ``pending`` (None, a tensor or a ``SideBySideOutput``).
+
+    * ``rows`` (int32): returns float x of those rows.
+    * ``raw``: returns x in ``act_dtype``.
+    * ``norm_weight``: returns (x float, n = rmsnorm(x) * norm_weight in ``act_dtype`` or None
+      unless ``normed``, n + (n' - n) * shift in ``act_dtype`` or None without ``shift``).  n' is
+      the token before's n; that of an entry's first token is in ``prev`` (float [slots, >=
+      width], a view with one row a slot), which takes the entry's last n.
+    """
+    _need_cuda(resid, rows, norm_weight, shift, prev)
+    assert resid.dtype == torch.float32 and resid.dim() == 2 and resid.is_contiguous()
+    tokens, width = resid.shape
+    y0 = y1 = f = w0 = w1 = None
+    branch_eps = 0.0
+    if isinstance(pending, SideBySideOutput):
+        f = pending.ffn
+        if isinstance(pending.mixer, MeanOfNorms):
+            (y0, y1), (w0, w1) = pending.mixer.branches, pending.mixer.weights
+            branch_eps = pending.mixer.eps
+        else:
+            y0 = pending.mixer
+    elif pending is not None:
+        y0 = pending.materialize() if hasattr(pending, "materialize") else pending
+    for t in (y0, y1, f):
+        if t is not None:
+            _need_cuda(t)
+            assert t.shape == resid.shape and t.is_contiguous()
+    act = act_dtype or next((t.dtype for t in (y1, f, y0) if t is not None), torch.float32)
+    for t in (y1, f):
+        assert t is None or t.dtype == act
+    assert y0 is None or y0.dtype in (act, torch.float32)
+    for w in (w0, w1):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == width)
+    dev = resid.device
+    x_out = raw_out = n_out = s_out = None
+    if rows is not None:
+        assert rows.dtype == torch.int32 and rows.is_contiguous()
+        x_out = torch.empty((rows.numel(), width), dtype=torch.float32, device=dev)
+    elif raw:
+        raw_out = torch.empty((tokens, width), dtype=act, device=dev)
+    else:
+        assert norm_weight is not None and norm_weight.numel() == width
+        x_out = torch.empty_like(resid) if y0 is not None else None
+        if normed:
+            n_out = torch.empty((tokens, width), dtype=act, device=dev)
+        if shift is not None:
+            assert shift.numel() == width and shift.dtype == norm_weight.dtype
+            assert prev.dtype == torch.float32 and prev.stride(1) == 1 and prev.shape[1] >= width
+            s_out = torch.empty((tokens, width), dtype=act, device=dev)
+    code = lib.get("side_by_side").mstar_side_step(
+        resid.data_ptr(), _ptr(y0), _dt(y0) if y0 is not None else F32, _ptr(y1), _ptr(f), _ptr(w0),
+        _ptr(w1), float(branch_eps), _ptr(x_out), _ptr(raw_out),
+        _ptr(norm_weight), _ptr(shift),
+        _dt(norm_weight) if norm_weight is not None else F32, float(eps), _ptr(n_out), _ptr(s_out),
+        _ptr(prev), prev.stride(0) if prev is not None else 0,
+        _ptr(ctx.token_req) if s_out is not None else 0,
+        _ptr(ctx.qo_indptr) if s_out is not None else 0, _ptr(ctx.slots) if s_out is not None else 0,
+        _ptr(rows), rows.numel() if rows is not None else 0, tokens, width, _DT[act], _stream())
+    if code == -1:
+        raise KernelError(f"side-by-side step refuses a width of {width}")
+    check(code, "side_step")
+    if rows is not None:
+        return x_out
+    if raw:
+        return raw_out
+    return (resid if x_out is None else x_out), n_out, s_out
+
+
+# ------------------------------------------------------------------ linear recurrences
+def _round4(n: int) -> int:
+    return -(-n // 4) * 4
+
+
+def time_mixing_state_size(width: int, heads: int, dim: int) -> int:
+    """Floats of one request's state: the last input row (padded to whole 16-byte pieces), then
+    S^T [heads, dim, dim]."""
+    return _round4(width) + heads * dim * dim
+
+
+def state_space_state_size(channels: int, taps: int, heads: int, n_state: int, vdim: int) -> int:
+    """Floats of one request's state: the convolution's last inputs [taps - 1, channels] (padded
+    to whole 16-byte pieces), then S^T [heads, vdim, n_state]."""
+    return _round4((taps - 1) * channels) + heads * n_state * vdim
+
+
+def time_mix(x: torch.Tensor, mu: torch.Tensor, ctx, state: torch.Tensor) -> torch.Tensor:
+    """[5, tokens, width]: x + (x' - x) * mu[s] for the five rows of ``mu`` (float), x' the
+    token before's row; that of an entry's first token comes from its slot (the first ``width``
+    floats of ``state``), which takes the entry's last row."""
+    _need_cuda(x, mu, state)
+    tokens, width = x.shape
+    assert x.stride(1) == 1 and mu.dtype == torch.float32 and mu.numel() == 5 * width
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= width
+    out = torch.empty((5, tokens, width), dtype=x.dtype, device=x.device)
+    check(lib.get("linear_recurrence").mstar_time_mix(
+        x.data_ptr(), x.stride(0), mu.data_ptr(), out.data_ptr(), ctx.token_req.data_ptr(),
+        ctx.qo_indptr.data_ptr(), ctx.slots.data_ptr(), state.data_ptr(), state.stride(0), _dt(x),
+        tokens, width, _stream()), "time_mix")
+    return out
+
+
+def tanh_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """tanh of float rows (a column view will do), in ``dtype``."""
+    _need_cuda(x)
+    assert x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1
+    out = torch.empty(tuple(x.shape), dtype=dtype, device=x.device)
+    check(lib.get("linear_recurrence").mstar_tanh_rows(
+        x.data_ptr(), x.stride(0), out.data_ptr(), _DT[dtype], x.shape[0], x.shape[1], _stream()),
+        "tanh_rows")
+    return out
+
+
+# tokens up to which the decay's second product is made inside ``mix_prepare``
+MIX_FUSED_TOKENS = 16
+
+
+def mix_prepare(rows: torch.Tensor, low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor,
+                u: torch.Tensor, heads: int, dim: int, dtype: torch.dtype):
+    """(decay float [tokens, heads * dim], direct float [tokens, heads]) of the time mixing:
+    ``decay = exp(-exp(W_w2 tanh(low) + w0))`` and ``direct = r . (u k)`` per head.  ``rows``:
+    float [tokens, >= 2 * heads * dim] with r and k side by side; ``low``: float [tokens, rank]
+    (a column view will do); ``w2`` [heads * dim, rank]; float ``w0``, ``u`` [heads * dim]."""
+    _need_cuda(rows, low, w2, w0, u)
+    tokens, hd = rows.shape[0], heads * dim
+    rank = w2.shape[1]
+    assert rows.dtype == torch.float32 and rows.stride(1) == 1 and rows.shape[1] >= 2 * hd
+    assert low.dtype == torch.float32 and tuple(low.shape) == (tokens, rank) and low.stride(1) == 1
+    assert w2.is_contiguous() and w2.shape[0] == hd
+    assert w0.dtype == torch.float32 and w0.numel() == hd and u.dtype == torch.float32 and u.numel() == hd
+    z = None
+    if tokens > MIX_FUSED_TOKENS or rank > 8192:
+        z = linear(tanh_rows(low, dtype), w2, out_dtype=torch.float32, static_weights=True)
+    decay = torch.empty((tokens, hd), dtype=torch.float32, device=rows.device)
+    direct = torch.empty((tokens, heads), dtype=torch.float32, device=rows.device)
+    check(lib.get("linear_recurrence").mstar_mix_prepare(
+        rows.data_ptr(), rows.stride(0), _ptr(z), hd, low.data_ptr(), low.stride(0), rank,
+        w2.data_ptr(), _dt(w2), w0.data_ptr(), u.data_ptr(), decay.data_ptr(), direct.data_ptr(),
+        tokens, heads, dim, _stream()), "mix_prepare")
+    return decay, direct
+
+
+def ssd_prepare(proj: torch.Tensor, conv_wt, conv_b, dt_bias, a_exp, ctx, state: torch.Tensor,
+                inner: int, channels: int, taps: int, heads: int):
+    """From the float projection [z | x | B | C | dt]: (silu(conv) of the x | B | C channels
+    [tokens, channels], dt [tokens, heads], decay = exp(-a_exp dt) [tokens, heads]), float.
+    ``conv_wt`` float [taps, channels], ``conv_b`` float [channels]; the rows before a portion
+    come from the slot ([taps - 1, channels] at its start), which ``linear_scan`` moves on."""
+    _need_cuda(proj, conv_wt, conv_b, dt_bias, a_exp, state)
+    tokens = proj.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1
+    assert proj.shape[1] == inner + channels + heads
+    assert tuple(conv_wt.shape) == (taps, channels) and conv_wt.is_contiguous()
+    for t, n in ((conv_wt, taps * channels), (conv_b, channels), (dt_bias, heads), (a_exp, heads)):
+        assert t.dtype == torch.float32 and t.numel() == n
+    assert state.dtype == torch.float32 and state.stride(1) == 1
+    dev = proj.device
+    xbc = torch.empty((tokens, channels), dtype=torch.float32, device=dev)
+    dt = torch.empty((tokens, heads), dtype=torch.float32, device=dev)
+    decay = torch.empty((tokens, heads), dtype=torch.float32, device=dev)
+    check(lib.get("linear_recurrence").mstar_ssd_prepare(
+        proj.data_ptr(), proj.stride(0), inner, channels, taps, heads, conv_wt.data_ptr(),
+        conv_b.data_ptr(), dt_bias.data_ptr(), a_exp.data_ptr(), ctx.token_req.data_ptr(),
+        ctx.qo_indptr.data_ptr(), ctx.slots.data_ptr(), state.data_ptr(), state.stride(0),
+        xbc.data_ptr(), dt.data_ptr(), decay.data_ptr(), tokens, _stream()), "ssd_prepare")
+    return xbc, dt, decay
+
+
+LINEAR_PIECE = 64           # fewest tokens of a piece of a scan that is cut into pieces
+
+
+def linear_scan_pieces(entries: int, heads: int, max_q_len: int, sms: int) -> tuple:
+    """(tokens of a piece or 0, pieces): entries are cut where they are long and the heads
+    alone leave most of the GPU idle, into as many pieces as give every SM some six blocks."""
+    forced = os.environ.get("MSTAR_LINEAR_PIECE")
+    if forced is not None:
+        piece = int(forced) // 16 * 16
+        return (piece, -(-max_q_len // piece)) if piece and max_q_len > piece else (0, 1)
+    blocks = max(entries * heads, 1)
+    want = min(-(-6 * sms // blocks), max_q_len // LINEAR_PIECE)
+    if want < 3:                                # two passes over the tokens: must pay
+        return 0, 1
+    piece = -(-(-(-max_q_len // want)) // 16) * 16
+    return piece, -(-max_q_len // piece)
+
+
+def linear_scan(r, k, v, decay, direct, ctx, state: torch.Tensor, offset: int, heads: int, dim: int,
+                vdim: int, *, vector_decay: bool, rk_share: int = 1, dt=None, raw=None,
+                channels: int = 0, taps: int = 0) -> torch.Tensor:
+    """The linear recurrence of a matrix state per head over the tokens of the step's entries,
+    each continuing the matrix S^T [heads, vdim, dim] at ``offset`` of its slot (updated in
+    place).  ``r``, ``k`` (heads / rk_share heads of ``dim``) and ``v`` (``heads`` of ``vdim``) are
+    float column views.
+
+    ``vector_decay``: ``decay`` [tokens, heads * dim]; o = S^T r + direct v with ``direct``
+    [tokens, heads], then S = diag(decay) S + k v^T.  Else ``decay`` [tokens, heads]; S = decay S
+    + k (dt v)^T with ``dt`` [tokens, heads], then o = S^T r + direct v with ``direct`` [heads].
+    ``raw``: rows whose first ``channels`` columns are a convolution's inputs; the slot's [taps -
+    1, channels] rows at its start move on.  Returns float [tokens, heads * vdim]."""
+    _need_cuda(r, k, v, decay, direct, dt, raw, state)
+    tokens = v.shape[0]
+    for t in (r, k, v):
+        assert t.dtype == torch.float32 and t.stride(1) == 1 and t.shape[0] == tokens
+    assert r.shape[1] == k.shape[1] == heads // rk_share * dim and v.shape[1] == heads * vdim
+    assert decay.dtype == torch.float32 and decay.is_contiguous()
+    assert tuple(decay.shape) == (tokens, heads * dim if vector_decay else heads)
+    assert direct.dtype == torch.float32 and direct.is_contiguous()
+    assert direct.numel() == (tokens * heads if vector_decay else heads)
+    assert dt is None or (dt.dtype == torch.float32 and tuple(dt.shape) == (tokens, heads))
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+    assert state.shape[1] >= offset + heads * dim * vdim
+    if taps > 1:
+        assert raw.dtype == torch.float32 and raw.stride(1) == 1 and raw.shape[1] >= channels
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=v.device)
+    entries = ctx.num_entries
+    piece, pieces = linear_scan_pieces(entries, heads, ctx.max_q_len, num_sms(v.device))
+    piece_state = piece_decay = None
+    if piece:
+        piece_state = torch.empty(entries * pieces * heads * vdim * dim, dtype=torch.float32,
+                                  device=v.device)
+        piece_decay = torch.empty(entries * pieces * heads * (dim if vector_decay else 1),
+                                  dtype=torch.float32, device=v.device)
+    code = lib.get("linear_recurrence").mstar_linear_scan(
+        r.data_ptr(), k.data_ptr(), v.data_ptr(), r.stride(0), k.stride(0), v.stride(0), rk_share,
+        decay.data_ptr(), int(vector_decay), direct.data_ptr(), _ptr(dt), ctx.qo_indptr.data_ptr(),
+        ctx.slots.data_ptr(), state.data_ptr(), state.stride(0), offset, out.data_ptr(), entries,
+        ctx.max_q_len, heads, dim, vdim, piece, pieces, _ptr(piece_state), _ptr(piece_decay),
+        _ptr(raw), raw.stride(0) if raw is not None else 0, channels, taps, _stream())
+    if code == -1:
+        raise KernelError(f"linear scan refuses heads={heads}, dim={dim}, vdim={vdim} (dim at most "
+                          "512)")
+    check(code, "linear_scan")
+    if piece:
+        lib.add_launches(2)                     # three kernels behind one call
     return out

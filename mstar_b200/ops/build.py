@@ -49,6 +49,8 @@ LIBRARIES = {
     "selective_scan": ("cuda", ["selective_scan.cu"], []),
     "gated_delta": ("cuda", ["gated_delta.cu"], []),
     "hyper": ("cuda", ["hyper.cu"], []),
+    "side_by_side": ("cuda", ["side_by_side.cu"], []),
+    "linear_recurrence": ("cuda", ["linear_recurrence.cu"], []),
     "host": ("host", ["host/cache_manager.cpp"], []),
 }
 

@@ -23,7 +23,7 @@ _SIGNATURES = {
         "mstar_scale_softcap": [_vp, _ll, _f, _f, _vp],
         "mstar_add_rmsnorm": [_vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _f, _i, _vp],
         "mstar_gather_add_rows": [_vp, _vp, _i, _vp, _vp, _i, _i, _vp],
-        "mstar_silu_mul": [_vp, _vp, _i, _i, _i, _i, _vp],
+        "mstar_silu_mul": [_vp, _vp, _i, _i, _i, _i, _f, _f, _vp],
         "mstar_convert": [_vp, _i, _vp, _i, _ll, _vp],
         "mstar_rope_kv_write": [_vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i,
                                 _i, _i, _vp],
@@ -55,7 +55,7 @@ _SIGNATURES = {
     "matrix_memory": {
         "mstar_matrix_memory_scan": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _i,
                                      _i, _i, _i, _f, _f, _f, _vp],
-        "mstar_head_norm_gate": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
+        "mstar_head_norm_gate": [_vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _vp],
     },
     "attention_latent": {
         "mstar_latent_attention": [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i,
@@ -64,11 +64,11 @@ _SIGNATURES = {
                               _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
     },
     "routed_experts": {
-        "mstar_route_topk": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+        "mstar_route_topk": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
         "mstar_experts_by_row": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                                 _i, _i, _vp],
+                                 _i, _i, _f, _f, _vp, _i, _vp],
         "mstar_experts_grouped": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
-                                  _i, _i, _i, _i, _vp],
+                                  _i, _i, _i, _i, _f, _f, _vp, _i, _vp],
     },
     "attention_sink": {
         "mstar_sink_prepare": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i,
@@ -76,11 +76,26 @@ _SIGNATURES = {
                                _vp, _ll, _i, _i, _f, _i, _vp],
         "mstar_conv_state_advance": [_vp, _i, _i, _i, _vp, _vp, _vp, _ll, _i, _vp],
         "mstar_sink_attention_generic": [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i,
-                                         _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp],
+                                         _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _i, _i, _vp, _vp],
     },
     "attention_sink_tc": {
         "mstar_sink_attention_tc": [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                                    _i, _i, _i, _i, _f, _i, _vp, _vp, _i, _i, _f, _vp, _vp],
+                                    _i, _i, _i, _i, _f, _i, _vp, _vp, _i, _i, _f, _vp, _i, _i, _vp,
+                                    _vp],
+    },
+    "side_by_side": {
+        "mstar_side_step": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _f, _vp,
+                            _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    },
+    "linear_recurrence": {
+        "mstar_time_mix": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _vp],
+        "mstar_tanh_rows": [_vp, _i, _vp, _i, _i, _i, _vp],
+        "mstar_mix_prepare": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i,
+                              _vp],
+        "mstar_ssd_prepare": [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll,
+                              _vp, _vp, _vp, _i, _vp],
+        "mstar_linear_scan": [_vp, _vp, _vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _ll,
+                              _ll, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _vp],
     },
     "selective_scan": {
         "mstar_conv_silu": [_vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i,
@@ -112,14 +127,17 @@ _SIGNATURES = {
         "mstar_sgemm_nt": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     },
     "gemm_smallm_bulk": {
-        "mstar_gemm_smallm_bulk_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp],
+        "mstar_gemm_smallm_bulk_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _f,
+                                        _vp],
+        "mstar_gemm_smallm_bulk_planes": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _ll, _i, _vp,
+                                          _vp],
         "mstar_gemm_smallm_bulk_relu2_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp],
         "mstar_qkv_rope_write_bulk_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i,
                                            _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp],
     },
     "gemm_tcgen05": {
         "mstar_gemm_tcgen05_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp],
-        "mstar_gemm_tcgen05_gated_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
+        "mstar_gemm_tcgen05_gated_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _f, _f, _vp],
     },
     "gemm_skinny": {
         "mstar_gemm_skinny_bf16": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp],

@@ -21,7 +21,9 @@ gate a head on the output; the gate's rows ride in the fused first product.  Fur
 options of that path: an RMS norm over the whole q (and k) projection instead of a head,
 rotary pairs of neighbouring features, a query temperature that grows with the logarithm of
 the position, a tanh soft cap on the scores, a sink in the softmax's denominator (a learned
-number a head, or zero), and a sigmoid gate a feature on the heads' outputs.
+number a head, or zero), a sigmoid gate a feature on the heads' outputs, a mask of chunks
+instead of a window (the cache then keeps as many keys as a chunk is long), a learned number
+a head added to the scores, and weights that are sigmoids of the scores instead of a softmax.
 """
 from __future__ import annotations
 
@@ -60,6 +62,8 @@ class Attention:
             first["k_norm.weight"] = ParamSpec((per_k * spec.head_dim,), role="vector", init="ones")
         if spec.sink == "learned":
             first["sink"] = ParamSpec((spec.num_heads,), role="vector", init="zeros")
+        if spec.score_bias:
+            first["score_bias"] = ParamSpec((spec.num_heads,), role="vector", init="zeros")
         if spec.conv_taps:
             first["q_conv.weight"] = ParamSpec((q_rows, spec.conv_taps), role="vector")
             first["k_conv.weight"] = ParamSpec((spec.num_kv_heads * spec.head_dim, spec.conv_taps),
@@ -74,7 +78,7 @@ class Attention:
             channels = (spec.num_heads + spec.num_kv_heads) * spec.head_dim
             state = StateNeed(shape=((spec.conv_taps - 1) * channels,), dtype="float32")
         return CacheNeed(kv=KVNeed(num_kv_heads=spec.num_kv_heads, head_dim=spec.head_dim,
-                                   window=spec.window, keep_first=spec.keep_first if spec.window
+                                   window=spec.chunk or spec.window, keep_first=spec.keep_first if spec.window
                                    else 0,
                                    v_head_dim=None if spec.value_dim == spec.head_dim
                                    else spec.value_dim), state=state)
@@ -110,6 +114,15 @@ class Attention:
             self.sink = params["sink"].float().contiguous()
         elif spec.sink == "zero":
             self.sink = torch.zeros(spec.num_heads, dtype=torch.float32, device=runtime.device)
+        if spec.weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"attention weights {spec.weights!r} are not known (softmax, sigmoid)")
+        if spec.weights == "sigmoid" and spec.sink is not None:
+            raise ValueError("a sink belongs to a softmax")
+        if spec.chunk and spec.window:
+            raise ValueError("an attention has a window or chunks, not both")
+        self.score_bias = None
+        if spec.score_bias:
+            self.score_bias = params["score_bias"].float().contiguous()
         small = [w for w in (self.bias, self.q_norm, self.k_norm, self.q_conv, self.k_conv)
                  if w is not None]
         if len({w.dtype for w in small}) > 1:   # the input kernel takes them in one type
@@ -123,8 +136,6 @@ class Attention:
             if p.kind not in ("rope", "none"):
                 raise ValueError("this attention rotates pairs of features (a rope position "
                                  "spec) or nothing")
-            if p.interleaved and p.scaling is not None:
-                raise ValueError("frequency scaling goes with split-half pairs here")
             self.rot = p.rotary_dim if p.kind == "rope" else 0
             self.freq = None
             if self.rot:
@@ -176,7 +187,8 @@ class Attention:
                                  s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim,
                                  cache.page_size, s.window or 0, s.keep_first if s.window else 0,
                                  self.scale, ctx=ctx, gate=gate, softcap=s.softcap,
-                                 sink=self.sink)
+                                 sink=self.sink, chunk=s.chunk or 0,
+                                 sigmoid=s.weights == "sigmoid", bias=self.score_bias)
         return ops.linear(out, self.w_out, static_weights=True)
 
     def attend(self, qkv, out, ctx: StepContext, cache: LayerCache) -> None:

@@ -113,6 +113,9 @@ class ResidualStream:
 
         if self.copies is not None:
             return self.copies.gather(rows)
+        if self.post is None and hasattr(self.delta, "gather"):    # adds itself on the way
+            d, self.delta = self.delta, None
+            return d.gather(self.h, rows)
         return ops.gather_add_rows(self.h, self.take_delta(), rows)
 
     def push(self, delta: torch.Tensor, post=None, scale: float = 1.0) -> None:
@@ -146,6 +149,19 @@ class ResidualStream:
             scale = self.post_scale
             d, post = self.take_pending()
             post.add_normed(self.h, d, scale)
+
+    def read_rows(self, dtype: torch.dtype) -> torch.Tensor:
+        """The residual with everything pending added, as new rows of ``dtype``; the stream's own
+        residual and what is pending stay as they are."""
+        from .. import ops
+
+        if self.copies is not None:
+            raise RuntimeError("a residual of several copies has no rows of its own")
+        if self.post is not None:
+            self.settle()
+        if self.delta is None:
+            return ops.convert(self.h, dtype)
+        return ops.side_step(self.h, self.delta, act_dtype=dtype, raw=True)
 
     def rows(self, dtype: torch.dtype) -> torch.Tensor:
         """The residual itself, everything pending added, as rows of ``dtype`` for a sublayer

@@ -7,10 +7,13 @@ passes: each part's output stays pending on the residual stream and the next nor
 """
 from __future__ import annotations
 
+import os
+from dataclasses import replace
+
 import torch
 
 from ..weights.names import ParamSpec
-from .base import ResidualStream, Runtime
+from .base import CacheNeed, ResidualStream, Runtime, StateNeed
 from .registry import build_part, part_class, register_part
 
 
@@ -276,7 +279,112 @@ class HyperBlock:
             copies.pending = self._pending(self.ffn.forward(y, ctx), 2)
 
 
+class SideBySideBlock:
+    """h += mixer(n~) + ffn(n) with one norm, n = norm1(h); with ``token_shift`` the mixer reads
+    n~ = n + (n' - n) * shift, n' the previous token's n, else n itself.  The two outputs stay
+    pending together; the next block's kernel adds them, norms and shifts at once, and writes the
+    new residual into a buffer of its own (the residual it reads is left as it is).  An entry's
+    last n follows the mixer's own state in the layer's state slot.
+
+    The sublayers do not depend on one another: the feed-forward runs on a stream of its own,
+    forked from and joined to the step's (MSTAR_PARALLEL_STREAMS=0: one after the other)."""
+
+    keeps_residual = True       # never writes into the residual tensor it is given
+
+    @staticmethod
+    def _subparts(spec):
+        parts = [("norm1", "norm"), ("mixer", "mixer")]
+        if spec.ffn is not None:
+            parts.append(("ffn", "ffn"))
+        return parts
+
+    @classmethod
+    def param_specs(cls, spec) -> dict:
+        out = {}
+        for name, category in cls._subparts(spec):
+            sub = getattr(spec, name)
+            if sub is None:
+                raise ValueError(f"a side-by-side block needs {name}")
+            for local, ps in part_class(category, sub).param_specs(sub).items():
+                out[f"{name}.{local}"] = ps
+        if spec.token_shift:
+            out["shift"] = ParamSpec((spec.norm1.size,), role="vector", init="zeros")
+        return out
+
+    @staticmethod
+    def _mixer_state(spec):
+        """(the mixer's cache need, floats of its state, padded to whole 16-byte pieces)"""
+        need = part_class("mixer", spec.mixer).cache_need(spec.mixer) or CacheNeed()
+        size = 0
+        if need.state is not None:
+            if need.state.dtype != "float32" or len(need.state.shape) != 1:
+                raise ValueError("a token shift shares its slot with a flat float state only")
+            size = -(-need.state.shape[0] // 4) * 4
+        return need, size
+
+    @classmethod
+    def cache_need(cls, spec):
+        if not spec.token_shift:
+            return part_class("mixer", spec.mixer).cache_need(spec.mixer)
+        need, size = cls._mixer_state(spec)
+        total = size + -(-spec.norm1.size // 4) * 4
+        return CacheNeed(kv=need.kv, state=StateNeed(shape=(total,), dtype="float32"))
+
+    def __init__(self, spec, params: dict, runtime: Runtime):
+        self.spec = spec
+        self.runtime = runtime
+        self.parts = {name: build_part(category, getattr(spec, name), _sub(params, name), runtime)
+                      for name, category in self._subparts(spec)}
+        self.norm1, self.mixer = self.parts["norm1"], self.parts["mixer"]
+        self.ffn = self.parts.get("ffn")
+        if self.norm1.spec.kind != "rmsnorm" or self.norm1.spec.weight_offset:
+            raise ValueError("a side-by-side block reads through a plain RMS norm")
+        self.shift = None
+        if spec.token_shift:
+            self.shift = params["shift"].to(self.norm1.weight.dtype).contiguous()
+            self.need, self.mixer_floats = self._mixer_state(spec)
+        self.graph_safe = all(getattr(p, "graph_safe", False) is True for p in self.parts.values())
+        self.side_stream = None
+        if self.ffn is not None and os.environ.get("MSTAR_PARALLEL_STREAMS") != "0":
+            self.side_stream = torch.cuda.Stream(device=runtime.device)
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> None:
+        from .. import ops
+
+        if stream.copies is not None:
+            raise ValueError("a side-by-side block works on one residual")
+        stream.settle()                          # a delta with a norm of its own came before
+        prev, mixer_cache = None, cache
+        if self.shift is not None:
+            prev = cache.state[:, self.mixer_floats:]
+            own = None
+            if self.need.state is not None:
+                own = cache.state[:, :self.need.state.shape[0]]
+            mixer_cache = replace(cache, state=own)
+        h, n, shifted = ops.side_step(
+            stream.h, stream.take_pending()[0], act_dtype=self.runtime.dtype,
+            norm_weight=self.norm1.weight, eps=self.norm1.spec.eps, shift=self.shift, prev=prev,
+            ctx=ctx, normed=self.ffn is not None or self.shift is None)
+        stream.h = h
+        x = n if shifted is None else shifted
+        f = None
+        if self.side_stream is None:
+            y = self.mixer.forward(x, ctx, mixer_cache)
+            if self.ffn is not None:
+                f = self.ffn.forward(n, ctx)
+        else:
+            main = torch.cuda.current_stream(self.runtime.device)
+            self.side_stream.wait_stream(main)
+            with torch.cuda.stream(self.side_stream):
+                f = self.ffn.forward(n, ctx)
+            y = self.mixer.forward(x, ctx, mixer_cache)
+            main.wait_stream(self.side_stream)
+            f.record_stream(main)
+        stream.push(ops.SideBySideOutput(y, f))
+
+
 register_part("block", "hyper", HyperBlock)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "postnorm", PostNormBlock)
 register_part("block", "sandwich", SandwichBlock)
+register_part("block", "side_by_side", SideBySideBlock)

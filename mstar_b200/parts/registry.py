@@ -25,7 +25,7 @@ and the step context.
 """
 from __future__ import annotations
 
-CATEGORIES = ("mixer", "ffn", "norm", "position", "block", "embedding", "head")
+CATEGORIES = ("mixer", "ffn", "norm", "position", "block", "embedding", "head", "loop_input")
 
 _PARTS: dict = {}
 
@@ -71,5 +71,5 @@ def _builtin() -> None:
         return
     _done = True
     from . import (attention, block, embedding, gated_delta, latent_attention,  # noqa: F401
-                   matrix_memory, mlp, norm, parallel, rope, routed_experts,
-                   selective_scan)   # (they register themselves)
+                   loop_input, matrix_memory, mlp, norm, parallel, rope, routed_experts,
+                   selective_scan, state_space, time_mixing)   # (they register themselves)

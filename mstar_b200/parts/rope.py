@@ -1,4 +1,4 @@
-"""Rotary position encoding with the llama3 frequency scaling.
+"""Rotary position encoding with the llama3 or the linear frequency scaling.
 
 Unscaled: inv_freq_j = theta^(-2j/rotary_dim), angle = position * inv_freq_j,
 (x1, x2) -> (x1 cos - x2 sin, x2 cos + x1 sin) on split-half pairs
@@ -11,6 +11,7 @@ wavelength L = 2 pi / inv_freq and original context C:
     L > C / low_freq_factor   -> inv_freq / factor
     otherwise s = (C / L - low) / (high - low),
               inv_freq' = (1 - s) * inv_freq / factor + s * inv_freq.
+The linear rule divides every frequency by the factor.
 The table of frequencies is computed once on the host in double precision and
 rounded to float; angles are float(position) * inv_freq in float on the device.
 """
@@ -32,6 +33,8 @@ def rope_inverse_frequencies(spec) -> list:
     sc = spec.scaling
     if sc is None:
         return freqs
+    if sc.rope_type == "linear":
+        return [f / sc.factor for f in freqs]
     if sc.rope_type != "llama3":
         raise ValueError(f"rope scaling {sc.rope_type!r} is not supported")
     low_wavelen = sc.original_max_position_embeddings / sc.low_freq_factor

@@ -4,7 +4,8 @@ feed-forwards per token; an optional shared one runs for every token and is adde
 The router's logits are a product with float output; a kernel turns them into the chosen
 experts and their weights (sigmoid or softmax scores, renormalised or not).  The shared
 expert is the dense gated feed-forward's path (one fused gate/up product, one down
-product); the routed experts' kernels add its output while they write theirs.  A few rows
+product); the routed experts' kernels add its output while they write theirs, times the
+sigmoid of a gate a token where it has one (a further row of the router's product).  A few rows
 (decoded tokens) each stream the matrices of their experts; many rows (prompt portions)
 are sorted by expert on the device and run as tiles on the tensor cores.
 """
@@ -25,7 +26,8 @@ class RoutedExperts:
     def param_specs(cls, spec) -> dict:
         e, ff, width = spec.num_experts, spec.expert_size, spec.hidden_size
         outputs = e + spec.identity_experts
-        out = {"router.weight": ParamSpec((outputs, width))}
+        # the shared expert's gate is the row after the router's
+        out = {"router.weight": ParamSpec((outputs + (1 if spec.shared_gate else 0), width))}
         if spec.choice_bias:
             out["router.correction"] = ParamSpec((outputs,), role="vector", init="zeros")
         if spec.gated:
@@ -39,9 +41,16 @@ class RoutedExperts:
         return out
 
     def __init__(self, spec, params: dict, runtime: Runtime):
-        if (spec.gated, spec.activation) not in ((True, "silu"), (False, "relu2")):
+        if (spec.gated, spec.activation) not in ((True, "silu"), (True, "clamped_swish"),
+                                                 (False, "relu2")):
             raise ValueError(f"routed experts with gated={spec.gated} and activation "
-                             f"{spec.activation!r} have no kernel (gated silu and plain relu2 have)")
+                             f"{spec.activation!r} have no kernel (gated silu, gated clamped_swish "
+                             "and plain relu2 have)")
+        if spec.shared_gate and not spec.shared_size:
+            raise ValueError("a gate on the shared expert needs a shared expert")
+        clamped = spec.activation == "clamped_swish"
+        self.clamp = (spec.limit, spec.swish_alpha) if clamped else None
+        self.shared_clamp = {"limit": spec.shared_limit, "alpha": spec.swish_alpha} if clamped else {}
         if spec.identity_experts and spec.scale_input:
             raise ValueError("identity experts go with weights on the experts' outputs")
         if spec.score not in ("sigmoid", "softmax"):
@@ -60,15 +69,20 @@ class RoutedExperts:
     def forward(self, x, ctx):
         s = self.spec
         logits = ops.linear(x, self.router, out_dtype=torch.float32, static_weights=True)
+        shared_gate = None
+        if s.shared_gate:
+            logits, shared_gate = logits[:, :-1], logits[:, -1:]
         chosen, weight = ops.route_topk(logits, s.top, softmax=s.score == "softmax",
                                         renormalize=s.renormalize, choice_bias=self.correction)
         shared = None
         if self.shared_gate_up is not None:
-            shared = ops.linear(ops.gated_up(x, self.shared_gate_up, static_weights=True),
+            shared = ops.linear(ops.gated_up(x, self.shared_gate_up, static_weights=True,
+                                             kind=s.activation, **self.shared_clamp),
                                 self.shared_down, static_weights=True)
         return ops.routed_experts(x, self.gate_up, self.down, chosen, weight, s.num_experts,
                                   s.expert_size, s.scale_input, add=shared, gated=s.gated,
-                                  identity=s.identity_experts)
+                                  identity=s.identity_experts, clamp=self.clamp,
+                                  add_gate=shared_gate)
 
 
 register_part("ffn", "routed_experts", RoutedExperts)
