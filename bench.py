@@ -5,7 +5,7 @@ one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--rounds R] [--page-size P]
                     [--impl ours|reference] [--workloads all|none|mixed64|long8]
-    python bench.py --arch tifosun|vudivik|relurax|mokotar [--arch-size small|medium]   (another architecture)
+    python bench.py --arch tifosun|vudivik|relurax|mokotar|sokalorn [--arch-size small|medium]   (another architecture)
 
 One JSON line on stdout.  ``value``: decoded tokens per second of the engine's step
 function plus greedy sampling, timed on the device with CUDA events: W warm-up steps, then
@@ -426,6 +426,8 @@ def arch_bench(args) -> int:
         return relurax_bench(args)
     if args.arch == "mokotar":
         return mokotar_bench(args)
+    if args.arch == "sokalorn":
+        return sokalorn_bench(args)
     pk = peaks()
     t_cfg, l_cfg = tifosun_sizes(args.arch_size)
     page, batch = args.page_size, args.batch
@@ -1213,6 +1215,302 @@ def mokotar_bench(args) -> int:
     return 0
 
 
+# ------------------------------------------------------------------ a fifth architecture
+def sokalorn_sizes(name: str) -> tuple:
+    """(Sokalorn config, Vudivik config, Llama config) at layer sizes that resemble a real
+    model's: an attention in chunks beside a time mixing, and a state-space layer, in turn;
+    clamped experts with a gated shared one in every layer.  The Vudivik beside it, the
+    closest decoder of this engine (an attention of the same kernel family beside a
+    recurrent scan, routed experts), and the Llama have the same width, depth, vocabulary,
+    heads and key/value heads."""
+    if name == "small":
+        width, depth, vocab = 1024, 8, 32000
+        heads, kv_heads, experts, top, ff, shared, rank = 8, 2, 16, 2, 512, 1024, 64
+    elif name == "medium":
+        width, depth, vocab = 2048, 12, 64000
+        heads, kv_heads, experts, top, ff, shared, rank = 16, 4, 32, 4, 512, 2048, 64
+    else:
+        raise ValueError(f"unknown size {name!r} (small, medium)")
+    par = {"left": dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5,
+                        softcap=30.0, mask={"size": 1024},
+                        rot={"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0}}),
+           "right": dict(heads=width // 64, dim=64, decay_rank=rank)}
+    ssd = dict(heads=2 * width // 64, vdim=64, state=128, groups=2, conv=4, norm_groups=2)
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top},
+           "expert": {"ff": ff, "limit": 7.0}, "shared": {"ff": shared, "limit": 7.0}}
+    layers = [{"type": "mamba2" if i % 2 else "parallel",
+               "mixer": json.loads(json.dumps(ssd if i % 2 else par)), "mlp": moe}
+              for i in range(depth)]
+    sokalorn = {"architecture": "Sokalorn", "width": width, "vocab": vocab, "norm": {"eps": 1e-6},
+                "layers": layers}
+    vudivik, _ = vudivik_sizes(name)
+    llama = dict(ORPHEUS_3B, num_hidden_layers=depth, hidden_size=width,
+                 num_attention_heads=heads, num_key_value_heads=kv_heads, head_dim=128,
+                 intermediate_size=top * ff + shared, vocab_size=vocab, tie_word_embeddings=False)
+    return sokalorn, vudivik, llama
+
+
+def sokalorn_bench(args) -> int:
+    """``--arch sokalorn``: prefill and decode throughput of the Sokalorn decoder (random
+    weights, bfloat16) beside the Vudivik and Llama decoders at equal size, through the same
+    step function; then its kernels alone at the sizes of one layer, each beside the like
+    kernel of the closest decoder (sigmoid attention in chunks: Vudivik's window attention;
+    its input kernel: Vudivik's; the two recurrences and their input kernels: Vudivik's
+    selective scan and convolution, and the delta-rule scan at the time mixing's sizes; the
+    clamped experts: Vudivik's; sum, norm and token shift: Vudivik's mean of norms and
+    post-norm), with what each has to move against the measured peaks.  One JSON line."""
+    import torch
+
+    from mstar_b200 import ops
+    from mstar_b200.parts.base import StepContext
+
+    pk = peaks()
+    s_cfg, v_cfg, l_cfg = sokalorn_sizes(args.arch_size)
+    page, batch = args.page_size, args.batch
+    out = {"arch": "Sokalorn", "size": args.arch_size, "batch": batch, "prompt_len": PROMPT_LEN,
+           "peaks": pk["source"], "models": {}, "kernels": {}}
+    _time_models(args, (("sokalorn", s_cfg), ("vudivik", v_cfg), ("llama", l_cfg)), out)
+
+    dev = "cuda:0"
+    g = torch.Generator(device=dev).manual_seed(0)
+
+    def rnd(*shape, scale=1.0):
+        return (scale * torch.randn(*shape, generator=g, device=dev)).to(torch.bfloat16)
+
+    def f32(*shape):
+        return torch.randn(*shape, generator=g, device=dev)
+
+    def i32(v):
+        return torch.tensor(v, dtype=torch.int32, device=dev)
+
+    def record(name, ms, nbytes=None, flops=None, **more):
+        row = {"ms": round(ms, 4)}
+        if nbytes is not None:
+            row["gbs"] = round(nbytes / ms / 1e6, 1)
+            row["frac_hbm"] = round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4)
+        if flops is not None:
+            row["tflops"] = round(flops / ms / 1e9, 2)
+            row["frac_bf16"] = round(flops / ms / 1e9 / pk["bf16_tflops"], 5)
+        row.update(more)
+        out["kernels"][name] = row
+
+    width = s_cfg["width"]
+    left, right = (s_cfg["layers"][0]["mixer"][k] for k in ("left", "right"))
+    ssd, moe = s_cfg["layers"][1]["mixer"], s_cfg["layers"][0]["mlp"]
+    H, G, hd, chunk = left["heads"], left["kv_heads"], left["dim"], left["mask"]["size"]
+    ctx_len = PROMPT_LEN
+    pages_per = -(-ctx_len // page)
+    for tokens, reqs, label in ((batch, batch, "decode"), (PROMPT_LEN, 1, "prefill")):
+        per = tokens // reqs
+        copies = 1 if label == "prefill" else max(1, -(-(160 << 20) // (reqs * ctx_len * G * hd * 4)))
+        caches = [rnd(reqs * pages_per + 1, 2, G, page, hd).view(reqs * pages_per + 1, -1)
+                  for _ in range(copies)]
+        table = torch.randperm(reqs * pages_per, device=dev).to(torch.int32).view(reqs, pages_per)
+        token_req = i32([r for r in range(reqs) for _ in range(per)])
+        cache_pos = i32([ctx_len - per + k for _ in range(reqs) for k in range(per)])
+        indptr = i32([k * per for k in range(reqs + 1)])
+        slots = i32(list(range(reqs)))
+        sc = StepContext(num_tokens=tokens, num_entries=reqs, token_req=token_req,
+                         positions=cache_pos, cache_pos=cache_pos, qo_indptr=indptr,
+                         kv_len=i32([ctx_len] * reqs), slots=slots, q_lens=[per] * reqs,
+                         kv_lens=[ctx_len] * reqs, host_slots=list(range(reqs)), max_q_len=per,
+                         max_kv_len=ctx_len, num_decode=reqs if per == 1 else 0)
+        reps = max(copies, 4) if label == "decode" else 2
+        turn = {"i": 0}
+
+        def rotated(items):
+            turn["i"] += 1
+            return items[turn["i"] % len(items)]
+
+        # attention and its input kernel
+        q, rows = rnd(tokens, H * hd), (H + 2 * G) * hd
+        qkv = f32(tokens, rows + H * hd)                        # [q | k | v | gate]
+        bias = f32(H)
+        ckeys = sum((ctx_len - per + k) % chunk + 1 for k in range(per)) * reqs
+        wkeys = sum(min(ctx_len - per + k + 1, 1024) + 4 for k in range(per)) * reqs
+        kv_bytes = G * hd * 4.0 * reqs
+        ms = _time_graph(lambda: ops.sink_attention(
+            q, rotated(caches), table, token_req, cache_pos, H, G, hd, hd, page, 0, 0, left["scale"],
+            ctx=sc, gate=qkv[:, rows:], softcap=left["softcap"], chunk=chunk, sigmoid=True, bias=bias),
+            reps=reps)
+        record(f"sigmoid_chunk_attention_{label}", ms, nbytes=kv_bytes * min(ctx_len, chunk if per == 1 else ctx_len),
+               flops=4.0 * H * ckeys * hd)
+        ms = _time_graph(lambda: ops.sink_attention(
+            q, rotated(caches), table, token_req, cache_pos, H, G, hd, hd, page, 1024, 4,
+            left["scale"], ctx=sc), reps=reps)
+        record(f"vudivik_window_attention_{label}", ms, nbytes=kv_bytes * min(ctx_len, 1028 if per == 1 else ctx_len),
+               flops=4.0 * H * wkeys * hd)
+        freq = torch.rand(32, dtype=torch.float64, device=dev)
+        freq_v = torch.rand(hd // 2, dtype=torch.float64, device=dev)
+        io_bytes = tokens * (rows * 4 + H * hd * 2 + 2 * G * hd * 2.0)
+        ms = _time_graph(lambda: ops.sink_prepare(
+            qkv, None, None, None, freq, cache_pos, cache_pos, token_req, table, caches[0], H, G, hd,
+            hd, 64, page, 0.0, torch.bfloat16), reps=8)
+        record(f"rope_cache_{label}", ms, nbytes=io_bytes)
+        vb, nq, nk = rnd(rows), rnd(hd), rnd(hd)
+        ms = _time_graph(lambda: ops.sink_prepare(
+            qkv, vb, nq, nk, freq_v, cache_pos, cache_pos, token_req, table, caches[0], H, G, hd, hd,
+            hd, page, 1e-6, torch.bfloat16), reps=8)
+        record(f"vudivik_bias_norm_rope_cache_{label}", ms, nbytes=io_bytes)
+
+        # time mixing
+        RH, D, rank = right["heads"], right["dim"], right["decay_rank"]
+        size = ops.time_mixing_state_size(width, RH, D)
+        n_state = max(1, -(-(160 << 20) // (reqs * size * 4))) if label == "decode" else 1
+        states = [torch.zeros(reqs, size, device=dev) for _ in range(n_state)]
+        x, mu = rnd(tokens, width), torch.rand(5 * width, device=dev)
+        ms = _time_graph(lambda: ops.time_mix(x, mu, sc, states[0]), reps=8)
+        record(f"time_mix_{label}", ms, nbytes=tokens * width * 12.0)
+        mixes = ops.time_mix(x, mu, sc, states[0])
+        w_in = rnd(4 * RH * D + rank, width, scale=0.03)
+        ms = _time_graph(lambda: ops.linear_planes(mixes, w_in, RH * D, static_weights=True), reps=8)
+        record(f"time_mixing_products_{label}", ms, nbytes=w_in.numel() * 2.0,
+               flops=2.0 * tokens * w_in.numel())
+        rkvg, low = ops.linear_planes(mixes, w_in, RH * D)
+        w2, w0, u = rnd(RH * D, rank), f32(RH * D) - 3.0, f32(RH * D)
+        ms = _time_graph(lambda: ops.mix_prepare(rkvg, low, w2, w0, u, RH, D, torch.bfloat16), reps=8)
+        record(f"time_mixing_decays_{label}", ms, nbytes=tokens * RH * D * 16.0)
+        decay, direct = ops.mix_prepare(rkvg, low, w2, w0, u, RH, D, torch.bfloat16)
+        r, k, v, gate = (rkvg[:, i * RH * D:(i + 1) * RH * D] for i in range(4))
+        offset = ops.time_mixing_state_size(width, 0, 0)
+        sreps = max(n_state, 4) if label == "decode" else 2
+        scan_bytes = lambda heads, d, vd, row: reqs * heads * d * vd * 8.0 + tokens * row * 4.0
+        ms = _time_graph(lambda: ops.linear_scan(r, k, v, decay, direct, sc, rotated(states), offset,
+                                                 RH, D, D, vector_decay=True), reps=sreps)
+        record(f"time_mixing_scan_{label}", ms, nbytes=scan_bytes(RH, D, D, 5 * RH * D),
+               tokens_per_us=round(per / ms / 1e3, 3), fp32_tflops=round(6.0 * tokens * RH * D * D / ms / 1e9, 2))
+        o, nw = f32(tokens, RH * D), f32(RH * D)
+        ms = _time_graph(lambda: ops.head_norm_gate(o, gate, nw, RH, D, 1e-6, torch.bfloat16, kind="silu"),
+                         reps=8)
+        record(f"time_mixing_norm_gate_{label}", ms, nbytes=tokens * RH * D * 10.0)
+
+        # state space
+        SH, VD, N, SG, taps = ssd["heads"], ssd["vdim"], ssd["state"], ssd["groups"], ssd["conv"]
+        inner = SH * VD
+        channels = inner + 2 * SG * N
+        size = ops.state_space_state_size(channels, taps, SH, N, VD)
+        n_state = max(1, -(-(160 << 20) // (reqs * size * 4))) if label == "decode" else 1
+        states2 = [torch.zeros(reqs, size, device=dev) for _ in range(n_state)]
+        proj = f32(tokens, inner + channels + SH)
+        cwt, cb = f32(taps, channels), f32(channels)
+        dtb, a_exp, skip = f32(SH) - 3.0, torch.rand(SH, device=dev) + 0.5, f32(SH)
+        prep = lambda: ops.ssd_prepare(proj, cwt, cb, dtb, a_exp, sc, states2[0], inner, channels, taps, SH)
+        ms = _time_graph(prep, reps=8)
+        record(f"state_space_conv_{label}", ms, nbytes=tokens * channels * 8.0)
+        xbc, dt, dec = prep()
+        offset2 = ops.state_space_state_size(channels, taps, 0, 0, 0)
+        sreps = max(n_state, 4) if label == "decode" else 2
+        ms = _time_graph(lambda: ops.linear_scan(
+            xbc[:, inner + SG * N:], xbc[:, inner:inner + SG * N], xbc[:, :inner], dec, skip, sc,
+            rotated(states2), offset2, SH, N, VD, vector_decay=False, rk_share=SH // SG, dt=dt,
+            raw=proj[:, inner:], channels=channels, taps=taps), reps=sreps)
+        record(f"state_space_scan_{label}", ms, nbytes=scan_bytes(SH, N, VD, 2 * inner + 2 * SG * N),
+               tokens_per_us=round(per / ms / 1e3, 3), fp32_tflops=round(6.0 * tokens * SH * N * VD / ms / 1e9, 2))
+        o, nw = f32(tokens, inner), f32(inner)
+        ms = _time_graph(lambda: ops.head_norm_gate(o, proj[:, :inner], nw, ssd["norm_groups"],
+                                                    inner // ssd["norm_groups"], 1e-6, torch.bfloat16,
+                                                    kind="silu", gate_first=True), reps=8)
+        record(f"state_space_gate_norm_{label}", ms, nbytes=tokens * inner * 10.0)
+
+        # like kernels: the delta-rule scan at the time mixing's sizes, its norm and gate;
+        # Vudivik's convolution and selective scan at its own
+        dq, dk, dv = f32(tokens, RH * D), f32(tokens, RH * D), f32(tokens, RH * D)
+        beta, dd = torch.rand(tokens, RH, device=dev), torch.rand(tokens, RH * D, device=dev)
+        dsize = ops.gated_delta_state_size(RH, RH, D, D, 1)
+        dstates = [torch.zeros(reqs, dsize, device=dev) for _ in range(
+            max(1, -(-(160 << 20) // (reqs * dsize * 4))) if label == "decode" else 1)]
+        ms = _time_graph(lambda: ops.delta_scan(dq, dk, dv, beta, dd, indptr, slots, rotated(dstates),
+                                                reqs, RH, RH, D, D, 1, max_q_len=per),
+                         reps=max(len(dstates), 4) if label == "decode" else 2)
+        record(f"mokotar_delta_scan_{label}", ms, nbytes=scan_bytes(RH, D, D, 5 * RH * D),
+               tokens_per_us=round(per / ms / 1e3, 3))
+        gb, nw1 = rnd(tokens, RH * D), f32(D)
+        ms = _time_graph(lambda: ops.delta_finish(dv, gb, nw1, RH, D, 1e-6, torch.bfloat16), reps=8)
+        record(f"mokotar_norm_gate_{label}", ms, nbytes=tokens * RH * D * 8.0)
+        vr = v_cfg["layers"][0]["mixer"]["right"]
+        vi, n_st, vrank, vt = vr["inner"], vr["state"], vr["dt_rank"], vr["conv"]
+        vsize = ops.selective_scan_state_size(vi, n_st, vt)
+        vstates = [torch.zeros(reqs, vsize, device=dev) for _ in range(
+            max(1, -(-(160 << 20) // (reqs * vsize * 4))) if label == "decode" else 1)]
+        xz, cw, cbv = rnd(tokens, 2 * vi), rnd(vi, vt), rnd(vi)
+        wt, bf = cw.float().t().contiguous(), cbv.float()
+        conv = lambda: ops.conv_silu(xz, cw, cbv, token_req, indptr, slots, vstates[0], vi, vt,
+                                     weight_t=wt, bias_f32=bf)
+        ms = _time_graph(conv, reps=8)
+        record(f"vudivik_conv_silu_{label}", ms, nbytes=tokens * vi * 4.0)
+        xc, vproj = conv(), f32(tokens, vrank + 2 * n_st)
+        w_dt, b_dt = f32(vi, vrank) * 0.1, f32(vi) - 4.0
+        a_neg, d_skip = -torch.rand(vi, n_st, device=dev) - 0.5, torch.ones(vi, device=dev)
+        ms = _time_graph(lambda: ops.selective_scan(xc, xz, vproj, w_dt, b_dt, a_neg, d_skip, indptr,
+                                                    slots, rotated(vstates), reqs, vi, n_st, vrank, vt,
+                                                    max_q_len=per),
+                         reps=max(len(vstates), 4) if label == "decode" else 2)
+        record(f"vudivik_selective_scan_{label}", ms,
+               nbytes=reqs * vi * n_st * 8.0 + tokens * (vi * 6 + (vrank + 2 * n_st) * 4.0),
+               tokens_per_us=round(per / ms / 1e3, 3), fp32_tflops=round(6.0 * tokens * vi * n_st / ms / 1e9, 2))
+
+        # experts, beside Vudivik's
+        E, top, ff, sff = (moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"],
+                           moe["shared"]["ff"])
+        copies = max(1, -(-(160 << 20) // (E * 3 * ff * width * 2)))
+        w_gu = [rnd(E * 2 * ff, width, scale=0.02) for _ in range(copies)]
+        w_dn = [rnd(E * width, ff, scale=0.02) for _ in range(copies)]
+        logits = f32(tokens, E + 1)
+        chosen, weight = ops.route_topk(logits[:, :E], top, softmax=True, renormalize=True)
+        add = rnd(tokens, width)
+
+        def experts():
+            i = turn["i"] = turn["i"] + 1
+            return ops.routed_experts(x, w_gu[i % copies], w_dn[i % copies], chosen, weight, E, ff, False,
+                                      add=add, clamp=(7.0, 1.702), add_gate=logits[:, E:])
+
+        ms = _time_graph(experts, reps=max(copies * 2, 4) if label == "decode" else 2)
+        used = len(set(chosen.flatten().tolist()))
+        record(f"clamped_experts_{label}", ms, nbytes=used * 3.0 * ff * width * 2,
+               flops=2.0 * tokens * top * 3 * ff * width, experts_used=used)
+        vm = v_cfg["layers"][1]["mlp"]
+        vE, vI, vtop, vff = (vm["router"]["experts"], vm["router"]["identity"], vm["router"]["top"],
+                             vm["expert"]["ff"])
+        w_up = [rnd(vE * vff, width, scale=0.02) for _ in range(copies)]
+        w_vd = [rnd(vE * width, vff, scale=0.02) for _ in range(copies)]
+        v_chosen, v_weight = ops.route_topk(f32(tokens, vE + vI), vtop, softmax=True,
+                                            choice_bias=torch.zeros(vE + vI, device=dev))
+
+        def v_experts():
+            i = turn["i"] = turn["i"] + 1
+            return ops.routed_experts(x, w_up[i % copies], w_vd[i % copies], v_chosen, v_weight, vE, vff,
+                                      False, gated=False, identity=vI)
+
+        ms = _time_graph(v_experts, reps=max(copies * 2, 4) if label == "decode" else 2)
+        picks = [e for e in v_chosen.flatten().tolist() if e < vE]
+        record(f"vudivik_experts_{label}", ms, nbytes=len(set(picks)) * 2.0 * vff * width * 2,
+               flops=2.0 * len(picks) * 2 * vff * width, experts_used=len(set(picks)))
+        w_sh = [rnd(2 * sff, width, scale=0.02) for _ in range(max(1, (160 << 20) // (4 * sff * width)))]
+        for kind in ("clamped_swish", "silu"):
+            ms = _time_graph(lambda: ops.gated_up(x, rotated(w_sh), static_weights=True, kind=kind,
+                                                  limit=7.0, alpha=1.702), reps=len(w_sh))
+            record(f"gated_up_{kind}_{label}", ms, nbytes=4.0 * sff * width,
+                   flops=4.0 * tokens * sff * width)
+
+        # between the layers, beside Vudivik's two kernels for the like
+        resid, ya, yb, f = f32(tokens, width), rnd(tokens, width), rnd(tokens, width), rnd(tokens, width)
+        wa, wb, nwt, shift = f32(width), f32(width), rnd(width), rnd(width)
+        prev = torch.zeros(reqs, width, device=dev)
+        pend = ops.SideBySideOutput(ops.MeanOfNorms([ya, yb], [wa, wb], 1e-6), f)
+        ms = _time_graph(lambda: ops.side_step(resid, pend, act_dtype=torch.bfloat16, norm_weight=nwt,
+                                               eps=1e-6, normed=True, shift=shift, prev=prev, ctx=sc),
+                         reps=20)
+        record(f"sum_norm_shift_{label}", ms, nbytes=tokens * width * (4 + 6 + 4 + 4.0))
+        mean = ops.MeanOfNorms([ya, yb], [wa, wb], 1e-6)
+        ms = _time_graph(lambda: ops.add_postnorm_rmsnorm(resid, mean, wa, 1e-6, 0.0,
+                                                          out_dtype=torch.bfloat16, post_scale=0.5,
+                                                          plain_out=True), reps=20)
+        record(f"vudivik_mean_postnorm_add_{label}", ms, nbytes=tokens * width * (4 + 4 + 4 + 2.0))
+    ops.check_error_word(dev)
+    print(json.dumps(out))
+    return 0
+
+
 # --------------------------------------------------------------- single kernels
 def _time_graph(fn, reps: int = 20, rounds: int = 5) -> float:
     """Median milliseconds of one call of ``fn`` when ``reps`` calls are replayed as one
@@ -1456,7 +1754,7 @@ def main() -> int:
     ap.add_argument("--small", action="store_true", help="a smaller case, for profiler captures")
     ap.add_argument("--sizes", default="orpheus-3b", choices=sorted(SIZES),
                     help="layer sizes; the default is the benchmark model")
-    ap.add_argument("--arch", default=None, choices=["tifosun", "vudivik", "relurax", "mokotar"],
+    ap.add_argument("--arch", default=None, choices=["tifosun", "vudivik", "relurax", "mokotar", "sokalorn"],
                     help="measure another architecture beside the Llama decoder at equal size "
                          "(prefill, decode, its own kernels) instead of the headline workload")
     ap.add_argument("--arch-size", default="small", choices=["small", "medium"])

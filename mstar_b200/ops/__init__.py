@@ -1788,7 +1788,7 @@ class SideBySideOutput:
         y = self.mixer.materialize() if hasattr(self.mixer, "materialize") else self.mixer
         return y if self.ffn is None else y.float() + self.ffn.float()
 
-    def gather(self, resid: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
+    def gather_rows(self, resid: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
         """float rows of ``resid`` plus this output."""
         return side_step(resid, self, rows=rows)
 

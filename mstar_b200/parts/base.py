@@ -113,9 +113,9 @@ class ResidualStream:
 
         if self.copies is not None:
             return self.copies.gather(rows)
-        if self.post is None and hasattr(self.delta, "gather"):    # adds itself on the way
+        if self.post is None and hasattr(self.delta, "gather_rows"):    # adds itself on the way
             d, self.delta = self.delta, None
-            return d.gather(self.h, rows)
+            return d.gather_rows(self.h, rows)
         return ops.gather_add_rows(self.h, self.take_delta(), rows)
 
     def push(self, delta: torch.Tensor, post=None, scale: float = 1.0) -> None:
