@@ -49,6 +49,8 @@ struct SinkTcArgs {
     const float* sink;          // null, or one number a query head
     int chunk;                  // 0: none
     const float* bias;          // null, or one number a query head
+    int span_tiles;             // > 0: row tiles of a span; the grid is a multiple of it
+    int fold;                   // > 0: from this rank on the order of the tiles is turned round
 };
 
 __device__ __forceinline__ float st_head_gate(const float* gate, int stride, int tok, int head) {
@@ -83,9 +85,25 @@ sink_attention_tc_kernel(SinkTcArgs a) {
     bf16* stages = reinterpret_cast<bf16*>(smem_raw);      // [NSTAGE]{K [64][LD], V [64][LD]}
     bf16* Qs = stages + NSTAGE * 2 * ST_TILE * LD;         // [64][LD]
 
-    const int split = blockIdx.x % a.splits;
-    const int tile = gridDim.x / a.splits - 1 - blockIdx.x / a.splits;   // long tiles first
-    const int kvh = blockIdx.y, e = blockIdx.z;
+    int split = blockIdx.x % a.splits;
+    int tile = gridDim.x / a.splits - 1 - blockIdx.x / a.splits;         // long tiles first
+    int kvh = blockIdx.y;
+    const int e = blockIdx.z;
+    if (a.span_tiles > 0) {
+        // one prompt: a tile's work grows with its place in its span (the chunk, or the prompt), so
+        // the tiles of all spans and heads are taken by that place, the last ones first; where all
+        // CTAs run at once, the second CTA of an SM comes from the other end (the one that shares
+        // its SM with the longest tile is the shortest)
+        const int tiles = gridDim.x / a.splits, n = tiles * a.nkv;
+        int rank = blockIdx.y * gridDim.x + blockIdx.x;
+        split = rank % a.splits;
+        rank /= a.splits;
+        if (a.fold > 0 && rank >= a.fold) rank = a.fold + n - 1 - rank;
+        const int same = tiles / a.span_tiles * a.nkv;         // tiles of one place
+        const int in_place = rank % same;
+        kvh = in_place % a.nkv;
+        tile = in_place / a.nkv * a.span_tiles + a.span_tiles - 1 - rank / same;
+    }
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int G = a.nq / a.nkv;
     const unsigned long long waited = pdl_wait();
@@ -454,7 +472,7 @@ __global__ void sink_merge_kernel(const float* __restrict__ scratch, bf16* __res
 }
 
 template <int D, int NSTAGE, bool KEYSPLIT, bool SIGMOID>
-static int launch_sink_tc_stages(const SinkTcArgs& a, int entries, int max_q_len, cudaStream_t s) {
+static int launch_sink_tc_stages(SinkTcArgs a, int entries, int max_q_len, cudaStream_t s) {
     const size_t smem = (size_t)(2 * NSTAGE + 1) * ST_TILE * (D + 8) * sizeof(bf16);
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
@@ -464,7 +482,18 @@ static int launch_sink_tc_stages(const SinkTcArgs& a, int entries, int max_q_len
         configured = true;
     }
     const int G = a.nq / a.nkv;
-    const long long tiles = ((long long)max_q_len * G + ST_ROWS - 1) / ST_ROWS;
+    long long tiles = ((long long)max_q_len * G + ST_ROWS - 1) / ST_ROWS;
+    a.span_tiles = a.fold = 0;
+    if (entries == 1 && tiles > 1) {
+        a.span_tiles = (int)tiles;
+        if (a.chunk > 0 && (long long)a.chunk * G / ST_ROWS < tiles) {
+            a.span_tiles = (int)((long long)a.chunk * G / ST_ROWS);
+            if (a.span_tiles < 1) a.span_tiles = 1;
+            tiles = (tiles + a.span_tiles - 1) / a.span_tiles * a.span_tiles;   // (tiles past the rows leave)
+        }
+        const int sms = device_sm_count();
+        if (a.splits == 1 && tiles * a.nkv > sms && tiles * a.nkv <= 2 * sms) a.fold = sms;
+    }
     if (tiles * a.splits > 2147483647LL) return -1;
     dim3 grid((unsigned)(tiles * a.splits), a.nkv, entries);
     mstar_launch((sink_attention_tc_kernel<D, NSTAGE, KEYSPLIT, SIGMOID>), grid, dim3(ST_THREADS), smem, s, a);

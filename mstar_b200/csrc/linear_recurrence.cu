@@ -10,8 +10,8 @@
 //                before an entry's first token comes from the slot, the entry's last row goes
 //                there (by the block that has read the slot).
 //   mix_prepare  decay = exp(-exp(z + w0)) per head and channel, z a product's float output or,
-//                for few tokens, made here as W_w2 tanh(low); and the current token's weight
-//                r . (u k) per head.
+//                for few tokens, made here as W_w2 tanh(low) (a block per token and head, eight
+//                lanes along a row of W_w2); and the current token's weight r . (u k) per head.
 //   ssd_prepare  causal convolution (bias) and SiLU of the x | B | C channels, dt = softplus(dt +
 //                bias), a = exp(-exp(A_log) dt).
 //   scan         below.
@@ -130,44 +130,65 @@ struct MixPrepArgs {
     int H, D;
 };
 
-// A block takes a token (and, of its heads, every gridDim.y-th set of warps); a warp a head.
-template <typename W>
-__global__ void __launch_bounds__(256) mix_prepare_kernel(MixPrepArgs a) {
-    extern __shared__ float low_s[];          // [rank]: tanh of the token's low row
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+// Many tokens: a warp per (token, head).
+__global__ void __launch_bounds__(128) mix_prepare_kernel(MixPrepArgs a, int pairs) {
+    const int lane = threadIdx.x & 31;
     const unsigned long long waited = pdl_wait();
+    const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (pair >= pairs) return;
+    const int t = pair / a.H, h = pair - t * a.H, hd = a.H * a.D;
     const float* row = pdl_after(a.rows, waited) + (size_t)t * a.ld;
-    const int hd = a.H * a.D;
-    if (a.z == nullptr) {
-        const float* low = pdl_after(a.low, waited) + (size_t)t * a.ld_low;
-        for (int i = threadIdx.x; i < a.rank; i += blockDim.x) low_s[i] = tanhf(low[i]);
-        __syncthreads();
+    const float* z = pdl_after(a.z, waited) + (size_t)t * a.ldz;
+    float sum = 0.f;
+    for (int d = lane; d < a.D; d += 32) {
+        const int i = h * a.D + d;
+        a.decay[(size_t)t * hd + i] = expf(-expf(z[i] + a.w0[i]));
+        sum = fmaf(row[i] * a.u[i], row[hd + i], sum);
     }
-    const float* z = pdl_after(a.z, waited);
+    sum = warp_sum(sum);
+    if (lane == 0) a.direct[(size_t)t * a.H + h] = sum;
+}
+
+// Few tokens: a block per (token, head); eight lanes take a row of W_w2, so that a warp reads
+// four whole rows at a time.
+template <typename W>
+__global__ void __launch_bounds__(128) mix_prepare_few_kernel(MixPrepArgs a) {
+    extern __shared__ float sm[];             // tanh of the token's low row [rank]
+    const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int sub = lane & 7, hd = a.H * a.D;
+    const unsigned long long waited = pdl_wait();
+    const float* low = pdl_after(a.low, waited) + (size_t)t * a.ld_low;
+    for (int i = threadIdx.x; i < a.rank; i += blockDim.x) sm[i] = tanhf(low[i]);
+    __syncthreads();
+    const float* row = pdl_after(a.rows, waited) + (size_t)t * a.ld + h * a.D;
     const bool vec = a.rank % 8 == 0 && ((uintptr_t)a.w2 & 15) == 0;
-    for (int h = blockIdx.y * nwarps + warp; h < a.H; h += nwarps * gridDim.y) {
-        float sum = 0.f;
-        for (int d = lane; d < a.D; d += 32) {
-            const int i = h * a.D + d;
-            float zi = 0.f;
-            if (a.z != nullptr) {
-                zi = z[(size_t)t * a.ldz + i];
-            } else {
-                const W* w = (const W*)a.w2 + (size_t)i * a.rank;
-                if (vec) {
-                    for (int c = 0; c < a.rank; c += 8) {
-                        float w8[8];
-                        load8(w + c, w8);
+    const W* w2 = (const W*)a.w2 + (size_t)h * a.D * a.rank;
+#pragma unroll 4
+    for (int d0 = warp * 4; d0 < a.D; d0 += (blockDim.x >> 5) * 4) {
+        const int d = d0 + (lane >> 3);
+        float z = 0.f;
+        if (d < a.D) {
+            const W* w = w2 + (size_t)d * a.rank;
+            if (vec) {
+                for (int c = sub * 8; c < a.rank; c += 64) {
+                    float w8[8];
+                    load8(w + c, w8);
 #pragma unroll
-                        for (int q = 0; q < 8; ++q) zi = fmaf(w8[q], low_s[c + q], zi);
-                    }
-                } else {
-                    for (int c = 0; c < a.rank; ++c) zi = fmaf(to_float(w[c]), low_s[c], zi);
+                    for (int q = 0; q < 8; ++q) z = fmaf(w8[q], sm[c + q], z);
                 }
+            } else {
+                for (int c = sub; c < a.rank; c += 8) z = fmaf(to_float(w[c]), sm[c], z);
             }
-            a.decay[(size_t)t * hd + i] = expf(-expf(zi + a.w0[i]));
-            sum = fmaf(row[i] * a.u[i], row[hd + i], sum);
         }
+        z += __shfl_xor_sync(0xffffffffu, z, 1);
+        z += __shfl_xor_sync(0xffffffffu, z, 2);
+        z += __shfl_xor_sync(0xffffffffu, z, 4);
+        if (sub == 0 && d < a.D)
+            a.decay[(size_t)t * hd + h * a.D + d] = expf(-expf(z + a.w0[h * a.D + d]));
+    }
+    if (warp == 0) {
+        float sum = 0.f;
+        for (int d = lane; d < a.D; d += 32) sum = fmaf(row[d] * a.u[h * a.D + d], row[hd + d], sum);
         sum = warp_sum(sum);
         if (lane == 0) a.direct[(size_t)t * a.H + h] = sum;
     }
@@ -181,19 +202,18 @@ MSTAR_API int mstar_mix_prepare(const float* rows, int ld, const float* z, int l
     if (H <= 0 || D <= 0 || ld < 2 * H * D) return -1;
     if (z == nullptr && (low == nullptr || w2 == nullptr || rank <= 0 || rank > 8192)) return -1;
     MixPrepArgs a{rows, ld, z, ldz, low, ld_low, rank, w2, w0, u, decay, direct, H, D};
-    const int warps = H < 8 ? H : 8;
-    int parts = 1;
-    if (tokens < device_sm_count()) {          // few tokens: a token's heads go to several blocks
-        parts = (H + warps - 1) / warps;
-        const int room = (2 * device_sm_count() + tokens - 1) / tokens;
-        if (parts > room) parts = room;
-    }
-    const size_t smem = z == nullptr ? sizeof(float) * rank : 0;
     cudaStream_t s = (cudaStream_t)stream;
+    if (z != nullptr) {
+        const int pairs = tokens * H;
+        mstar_launch(mix_prepare_kernel, dim3((pairs + 3) / 4), dim3(128), 0, s, a, pairs);
+        return launch_status();
+    }
+    if (H > 65535) return -1;
+    const size_t smem = sizeof(float) * rank;
     if (w2_dtype == MSTAR_F32)
-        mstar_launch((mix_prepare_kernel<float>), dim3(tokens, parts), dim3(32 * warps), smem, s, a);
+        mstar_launch((mix_prepare_few_kernel<float>), dim3(tokens, H), dim3(128), smem, s, a);
     else
-        mstar_launch((mix_prepare_kernel<bf16>), dim3(tokens, parts), dim3(32 * warps), smem, s, a);
+        mstar_launch((mix_prepare_few_kernel<bf16>), dim3(tokens, H), dim3(128), smem, s, a);
     return launch_status();
 }
 
@@ -398,35 +418,43 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(ScanArgs a) {
     auto fetch = [&](int buf, int base) {
         const int here = min(a.chunk, n - base);
         float* dst0 = stage + (size_t)buf * a.chunk * per_tok;
+        // a thread takes a piece of a token's rows (k, then decays, then r, then the values) and
+        // copies it for every token of the chunk: its addresses move on by fixed steps
         const int unit = VEC ? 4 : 1, per_row = D / unit;
-        const int per = (VECDECAY ? 3 : 2) * per_row;
-        // copy i of the chunk is piece p of token j; both move on by fixed steps
-        const int dj = threads / per, dp = threads % per;
-        int j = tid / per, p = tid % per;
-        for (; j < here; j += dj, p += dp) {
-            if (p >= per) { p -= per; ++j; if (j >= here) break; }
-            const int which = p / per_row, d = (p - which * per_row) * unit;
-            const size_t tok = (size_t)(start + base + j);
-            if (!OUT && which == 0) continue;             // no read-out
-            const float* src = which == 0 ? r + tok * a.ld_r + d
-                             : which == 1 ? k + tok * a.ld_k + d
-                                          : decay + (tok * a.H + h) * D + d;
-            float* dst = dst0 + (size_t)j * per_tok + which * DP + d;
-            if constexpr (VEC) lr_copy16(dst, src); else lr_copy4(dst, src);
+        const int all_rows = ((VECDECAY ? 2 : 1) + (OUT ? 1 : 0)) * per_row;
+        const int pieces_tok = all_rows + ncols / unit;
+        const size_t tok = (size_t)(start + base);
+        for (int p = tid; p < pieces_tok; p += threads) {
+            const float* src;
+            float* dst = dst0;
+            size_t step;
+            if (p >= all_rows) {
+                const int c = (p - all_rows) * unit;
+                src = v + tok * a.ld_v + col0 + c;
+                step = a.ld_v;
+                dst += (VECDECAY ? 3 : 2) * DP + c;
+            } else {
+                const int which = p / per_row, d = (p - which * per_row) * unit;
+                if (which == 0) {
+                    src = k + tok * a.ld_k + d;
+                    step = a.ld_k;
+                    dst += DP + d;
+                } else if (VECDECAY && which == 1) {
+                    step = (size_t)a.H * D;
+                    src = decay + tok * step + (size_t)h * D + d;
+                    dst += 2 * DP + d;
+                } else {
+                    src = r + tok * a.ld_r + d;
+                    step = a.ld_r;
+                    dst += d;
+                }
+            }
+#pragma unroll 4
+            for (int j = 0; j < here; ++j, src += step, dst += per_tok) {
+                if constexpr (VEC) lr_copy16(dst, src); else lr_copy4(dst, src);
+            }
         }
         float* vdst = dst0 + (VECDECAY ? 3 : 2) * DP;
-        if (VEC) {
-            const int q = ncols / 4;
-            for (int i = tid; i < here * q; i += threads) {
-                const int t = i / q, c = (i - t * q) * 4;
-                lr_copy16(vdst + (size_t)t * per_tok + c, v + (size_t)(start + base + t) * a.ld_v + col0 + c);
-            }
-        } else {
-            for (int i = tid; i < here * ncols; i += threads) {
-                const int t = i / ncols, c = i - t * ncols;
-                lr_copy4(vdst + (size_t)t * per_tok + c, v + (size_t)(start + base + t) * a.ld_v + col0 + c);
-            }
-        }
         for (int t = tid; t < here; t += threads) {
             const size_t at = (size_t)(start + base + t) * a.H + h;
             float* sc = vdst + (size_t)t * per_tok + cols;

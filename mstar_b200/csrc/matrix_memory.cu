@@ -287,8 +287,8 @@ MSTAR_API int mstar_matrix_memory_scan(const void* qkv, int act_dtype, int ld, i
 
 // out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * weight[h, :] * act(gate[t, h, :]), act the
 // sigmoid or (silu 1) the SiLU; with gate_first o act(gate) is normed and scaled.  One warp per
-// (token, head) where there are many, a block of four warps where there are few or the parts
-// are long; float sums.
+// (token, head) where there are many, a block where there are few or the parts are long; float
+// sums.
 __device__ __forceinline__ float hn_gate(float g, int silu) { return (silu ? g : 1.f) / (1.f + expf(-g)); }
 
 template <typename A, typename G, bool BLOCK>
@@ -325,10 +325,12 @@ MSTAR_API int mstar_head_norm_gate(const float* o, const void* gate, int gate_dt
     if (act_dtype == MSTAR_F32 && gate_dtype != MSTAR_F32) return -1;
     cudaStream_t s = (cudaStream_t)stream;
     const int pairs = tokens * heads, warps = 4;
-    const bool few = pairs < 4 * device_sm_count() || vdim >= 1024;
+    const bool scarce = pairs < 4 * device_sm_count(), few = scarce || vdim >= 1024;
+    // few long parts take more threads
+    const int threads = scarce && vdim >= 512 ? (vdim >= 1024 ? 512 : 256) : 32 * warps;
     dim3 grid(few ? pairs : (pairs + warps - 1) / warps);
 #define LAUNCH(A, G, B)                                                                           \
-    mstar_launch((head_norm_gate_kernel<A, G, B>), grid, dim3(32 * warps), 0, s, o, (const G*)gate, ldg, \
+    mstar_launch((head_norm_gate_kernel<A, G, B>), grid, dim3(threads), 0, s, o, (const G*)gate, ldg, \
                  weight, (A*)out, pairs, heads, vdim, eps, silu, gate_first)
     if (act_dtype == MSTAR_F32) {
         if (few) LAUNCH(float, float, true); else LAUNCH(float, float, false);

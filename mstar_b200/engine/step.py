@@ -99,7 +99,8 @@ class DecodeGraph:
             qo_indptr=view("qo_indptr"), kv_len=view("kv_len"), slots=view("slots"),
             q_lens=[1] * bucket, kv_lens=[bound] * bucket,
             host_slots=[storage.pad_slot] * bucket, max_q_len=1, max_kv_len=bound,
-            num_decode=bucket, token_source=(view("token_src"), stepper.device_tokens))
+            num_decode=bucket, token_source=(view("token_src"), stepper.device_tokens),
+            extras={"captured": True})
         self.tables = [view(f"table{g}").view(bucket, -1) for g in range(len(mgr.groups))]
         self.token_ids = view("token_ids")
         self.want_rows = view("want_rows")

@@ -1441,6 +1441,13 @@ def sink_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table, token_r
             max_keys = min(max_keys, chunk + ctx.max_q_len)
         splits = sink_attention_splits(ctx.num_entries, ctx.max_q_len, num_heads, num_kv_heads,
                                        max_keys, num_sms(q.device), wide=max(head_dim, v_dim))
+        if chunk and splits == 1 and ctx.num_entries == 1 and min(chunk, ctx.max_kv_len) >= 1024:
+            # one prompt whose CTAs all run at once: its time is that of the longest one, twice
+            # the mean, so the keys are shared between two (0.116 -> 0.087 ms for 2,048 tokens in
+            # chunks of 1,024; with more CTAs than run at once, or short chunks, it costs time)
+            row_tiles = -(-ctx.max_q_len * (num_heads // num_kv_heads) // 64) * num_kv_heads
+            if row_tiles <= 2 * num_sms(q.device):
+                splits = 2
         scratch = None
         if splits > 1:
             scratch = torch.empty(tokens * num_heads * splits * (v_dim + 2), dtype=torch.float32,
@@ -1964,7 +1971,7 @@ def ssd_prepare(proj: torch.Tensor, conv_wt, conv_b, dt_bias, a_exp, ctx, state:
     return xbc, dt, decay
 
 
-LINEAR_PIECE = 64           # fewest tokens of a piece of a scan that is cut into pieces
+LINEAR_PIECE = 32           # fewest tokens of a piece of a scan that is cut into pieces
 
 
 def linear_scan_pieces(entries: int, heads: int, max_q_len: int, sms: int) -> tuple:

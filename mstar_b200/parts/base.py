@@ -2,6 +2,7 @@
 residual stream and the description of a mixer's cache needs."""
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass, field
 from typing import Optional
 
@@ -46,6 +47,43 @@ class Runtime:
 
     dtype: torch.dtype
     device: torch.device
+
+
+class SideStream:
+    """A stream beside the step's own for work that does not depend on what the step's stream
+    does meanwhile: ``fork()`` is a context in which launches go there, ordered after what the
+    step's stream has been given so far; ``join(t)`` orders the step's stream after it (``t``:
+    what was made there and is used on the step's stream from here on).  In a captured step the
+    two become parallel branches of the graph.
+
+    A fork and its join cost the host some 0.1 ms of launches, so that outside a captured step
+    they pay where the step is long on the device (``wanted``); MSTAR_PARALLEL_STREAMS=0: never,
+    1: always."""
+
+    MIN_ELEMENTS = 4 << 20      # tokens x width of an uncaptured step from which on to fork
+
+    def __init__(self, device: torch.device):
+        self.device = device
+        self._forced = os.environ.get("MSTAR_PARALLEL_STREAMS")
+        self.stream = torch.cuda.Stream(device=device)
+        self._forked, self._done = torch.cuda.Event(), torch.cuda.Event()
+
+    def wanted(self, ctx: "StepContext", width: int) -> bool:
+        if self._forced in ("0", "1"):
+            return self._forced == "1"
+        return bool(ctx.extras.get("captured")) or ctx.num_tokens * width >= self.MIN_ELEMENTS
+
+    def fork(self):
+        self.main = torch.cuda.current_stream(self.device)
+        self._forked.record(self.main)
+        self.stream.wait_event(self._forked)
+        return torch.cuda.stream(self.stream)
+
+    def join(self, *made: torch.Tensor) -> None:
+        self._done.record(self.stream)
+        self.main.wait_event(self._done)
+        for t in made:
+            t.record_stream(self.main)
 
 
 @dataclass

@@ -7,13 +7,12 @@ passes: each part's output stays pending on the residual stream and the next nor
 """
 from __future__ import annotations
 
-import os
 from dataclasses import replace
 
 import torch
 
 from ..weights.names import ParamSpec
-from .base import CacheNeed, ResidualStream, Runtime, StateNeed
+from .base import CacheNeed, ResidualStream, Runtime, SideStream, StateNeed
 from .registry import build_part, part_class, register_part
 
 
@@ -287,7 +286,7 @@ class SideBySideBlock:
     last n follows the mixer's own state in the layer's state slot.
 
     The sublayers do not depend on one another: the feed-forward runs on a stream of its own,
-    forked from and joined to the step's (MSTAR_PARALLEL_STREAMS=0: one after the other)."""
+    forked from and joined to the step's, where that pays (``SideStream``)."""
 
     keeps_residual = True       # never writes into the residual tensor it is given
 
@@ -344,9 +343,7 @@ class SideBySideBlock:
             self.shift = params["shift"].to(self.norm1.weight.dtype).contiguous()
             self.need, self.mixer_floats = self._mixer_state(spec)
         self.graph_safe = all(getattr(p, "graph_safe", False) is True for p in self.parts.values())
-        self.side_stream = None
-        if self.ffn is not None and os.environ.get("MSTAR_PARALLEL_STREAMS") != "0":
-            self.side_stream = torch.cuda.Stream(device=runtime.device)
+        self.side_stream = SideStream(runtime.device) if self.ffn is not None else None
 
     def forward(self, stream: ResidualStream, ctx, cache) -> None:
         from .. import ops
@@ -368,18 +365,15 @@ class SideBySideBlock:
         stream.h = h
         x = n if shifted is None else shifted
         f = None
-        if self.side_stream is None:
+        if self.side_stream is None or not self.side_stream.wanted(ctx, x.shape[1]):
             y = self.mixer.forward(x, ctx, mixer_cache)
             if self.ffn is not None:
                 f = self.ffn.forward(n, ctx)
         else:
-            main = torch.cuda.current_stream(self.runtime.device)
-            self.side_stream.wait_stream(main)
-            with torch.cuda.stream(self.side_stream):
+            with self.side_stream.fork():
                 f = self.ffn.forward(n, ctx)
             y = self.mixer.forward(x, ctx, mixer_cache)
-            main.wait_stream(self.side_stream)
-            f.record_stream(main)
+            self.side_stream.join(f)
         stream.push(ops.SideBySideOutput(y, f))
 
 

@@ -9,17 +9,16 @@ and at most one a state slot: the layer's cache entry then serves both.
 The branches do not depend on one another, so each after the first runs on a stream of its
 own, forked from and joined to the stream of the step (in a captured decode step they become
 parallel branches of the graph): the short kernels of one branch fill the gaps between those
-of the other.  MSTAR_PARALLEL_STREAMS=0 runs them one after the other.
+of the other.  A step that is short on the device and not captured runs them one after the
+other (``SideStream``).
 """
 from __future__ import annotations
-
-import os
 
 import torch
 
 from .. import ops
 from ..weights.names import ParamSpec
-from .base import CacheNeed, LayerCache, Runtime, StepContext
+from .base import CacheNeed, LayerCache, Runtime, SideStream, StepContext
 from .registry import build_part, part_class, register_part
 
 
@@ -71,27 +70,19 @@ class ParallelMixer:
         self.weights = [params[f"out{b}.weight"].float().contiguous()
                         for b in range(len(spec.branches))] if spec.merge == "mean_of_norms" else []
         self.graph_safe = all(getattr(p, "graph_safe", False) is True for p in self.branches)
-        self.side_streams = None
-        if len(self.branches) > 1 and os.environ.get("MSTAR_PARALLEL_STREAMS") != "0":
-            self.side_streams = [torch.cuda.Stream(device=runtime.device)
-                                 for _ in self.branches[1:]]
+        self.side_streams = [SideStream(runtime.device) for _ in self.branches[1:]]
 
     def forward(self, x, ctx: StepContext, cache: LayerCache):
-        if self.side_streams is None:
+        if not self.side_streams or not self.side_streams[0].wanted(ctx, x.shape[1]):
             outs = [branch.forward(x, ctx, cache) for branch in self.branches]
             return self._merge(outs)
-        main = torch.cuda.current_stream(self.runtime.device)
         outs = [None] * len(self.branches)
         for b, side in enumerate(self.side_streams, start=1):
-            side.wait_stream(main)                       # x is ready there
-            with torch.cuda.stream(side):
+            with side.fork():                            # x is ready there
                 outs[b] = self.branches[b].forward(x, ctx, cache)
         outs[0] = self.branches[0].forward(x, ctx, cache)
-        for side in self.side_streams:
-            main.wait_stream(side)
-        # what the side streams allocated is used on the step's stream from here on
-        for out in outs[1:]:
-            out.record_stream(main)
+        for out, side in zip(outs[1:], self.side_streams):
+            side.join(out)
         return self._merge(outs)
 
     def _merge(self, outs):

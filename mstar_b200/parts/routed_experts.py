@@ -58,6 +58,10 @@ class RoutedExperts:
         self.spec = spec
         self.runtime = runtime
         self.router = params["router.weight"]
+        self.outputs = spec.num_experts + spec.identity_experts
+        if self.router.shape[0] % 8:            # whole 16-byte rows of logits for the product
+            pad = -self.router.shape[0] % 8
+            self.router = torch.cat([self.router, self.router.new_zeros((pad, spec.hidden_size))])
         self.gate_up = params["experts.gate_up.weight" if spec.gated else "experts.up.weight"]
         self.correction = None
         if spec.choice_bias:
@@ -69,9 +73,8 @@ class RoutedExperts:
     def forward(self, x, ctx):
         s = self.spec
         logits = ops.linear(x, self.router, out_dtype=torch.float32, static_weights=True)
-        shared_gate = None
-        if s.shared_gate:
-            logits, shared_gate = logits[:, :-1], logits[:, -1:]
+        shared_gate = logits[:, self.outputs:self.outputs + 1] if s.shared_gate else None
+        logits = logits[:, :self.outputs]
         chosen, weight = ops.route_topk(logits, s.top, softmax=s.score == "softmax",
                                         renormalize=s.renormalize, choice_bias=self.correction)
         shared = None

@@ -173,6 +173,27 @@ def test_attention_alone(dtype, m, page):
     close(torch.cat(outs), want, dtype, ("attention", m), bf16=3e-2)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("chunk,heads,kv_heads", [(1100, 8, 2), (300, 8, 2), (37, 8, 2), (2000, 16, 4), (None, 8, 2)])
+def test_long_prompts(dtype, chunk, heads, kv_heads):
+    """A prompt of two thousand tokens in one portion and as a short portion before a long one:
+    the order in which row tiles are taken, and the two shares of a long chunk's keys."""
+    m = U.left(heads, kv_heads, 16, 16, scale=0.25, softcap=5.0, chunk=chunk, rot_dims=8, base=5000.0)
+    part, spec, p = left_part(m, 64, dtype, seed=7)
+    T = 2100
+    x = rnd(T, 64, seed=8)
+    want = plain_left(x.double().numpy(), p, m)
+    for cuts in ([T], [37, T - 37]):
+        cache = paged_cache(spec, T, 16, dtype)
+        outs, at = [], 0
+        for n in cuts:
+            outs.append(part.forward(dev(x[at:at + n], dtype), step_ctx([n], [at]), cache))
+            at += n
+        err = (torch.cat(outs).double().cpu() - torch.from_numpy(want)).abs().amax(1)
+        err /= torch.from_numpy(want).abs().amax(1)
+        assert float(err.max()) < (1e-4 if dtype == "float32" else 5e-2), (cuts, int(err.argmax()), float(err.max()))
+
+
 def marked_inputs(p, m, width, T, marked, queries, gain=6.0):
     """Inputs in which the key at ``marked`` stands out for the ``queries``: the query tokens lie
     along a direction d, the marked token along the direction whose key equals the query of d (a
@@ -568,7 +589,7 @@ def test_mixed_batches_reuse_pages_and_slots(mixed_model, dtype, streams, monkey
     the sublayers on streams of their own and one after the other."""
     monkeypatch.setenv("MSTAR_PARALLEL_STREAMS", streams)
     weights, reqs, want, get = mixed_model
-    model = get(dtype) if streams == "1" else U.load(U.MIXED, weights, dtype)
+    model = U.load(U.MIXED, weights, dtype)
     schedule = [
         [("a", 2), ("b", 3), ("c", 1)],               # c ends here: its slot goes to d
         [("a", 29), ("b", 1), ("d", 16)],

@@ -131,7 +131,7 @@ def test_pieces_of_a_scan():
     assert linear_scan_pieces(8, 16, 1, 148) == (0, 1)            # decoding
     assert linear_scan_pieces(64, 32, 4096, 148) == (0, 1)        # the heads alone fill the GPU
     piece, pieces = linear_scan_pieces(1, 16, 2048, 148)
-    assert piece % 16 == 0 and piece >= 64 and (pieces - 1) * piece < 2048 <= pieces * piece
+    assert piece % 16 == 0 and piece >= 32 and (pieces - 1) * piece < 2048 <= pieces * piece
 
 
 def test_plain_mechanisms_on_hand_computed_cases():
