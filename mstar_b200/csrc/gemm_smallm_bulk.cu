@@ -64,10 +64,15 @@ __device__ __forceinline__ void sb_arrive(uint32_t bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
 }
 
-// the forms of the kernel; the last two have two 8 NT-row groups per strip
+// the forms of the kernel; those that sb_two_groups names have two 8 NT-row groups per strip
 #define SB_PLAIN 0
 #define SB_GATED 1
 #define SB_ROPE 2
+#define SB_CLAMPED 3                     // gated by the clamped swish
+#define SB_PLANES 4                      // plain, with several planes of x
+__host__ __device__ constexpr bool sb_two_groups(int mode) {
+    return mode == SB_GATED || mode == SB_ROPE || mode == SB_CLAMPED;
+}
 
 // what the rotary form needs beside the product's operands
 struct SbRope {
@@ -80,10 +85,10 @@ struct SbRope {
     int nq, nkv, hd, page_size, bt_stride;
     // plain form: 1 squares the positive part of every sum before it is stored (a
     // feed-forward's first product with its relu-squared, as one kernel); gated form: 0 gates
-    // by the SiLU, 2 by the tanh form of gelu, 3 by the clamped swish with limit and alpha
+    // by the SiLU, 2 by the tanh form of gelu
     int act;
-    float limit, alpha;
-    // plain form with plane_rows > 0: output features [p plane_rows, (p + 1) plane_rows) are
+    float limit, alpha;         // of the clamped form
+    // planes form: output features [p plane_rows, (p + 1) plane_rows) are
     // products with the rows of plane p of x, plane_stride elements apart (the last plane, planes
     // - 1, takes what is left)
     int plane_rows, planes;
@@ -109,11 +114,11 @@ __device__ __forceinline__ int sb_strip_n0(int strip, const SbRope& rp) {
 }
 
 template <int MODE, bool M16, int NT, typename OutT>
-__global__ void __launch_bounds__(SB_THREADS, (MODE ? 2 : 4) / NT >= 1 ? (MODE ? 2 : 4) / NT : 1)
+__global__ void __launch_bounds__(SB_THREADS, (sb_two_groups(MODE) ? 2 : 4) / NT >= 1 ? (sb_two_groups(MODE) ? 2 : 4) / NT : 1)
 smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT* __restrict__ out, int M,
                    int n_out, int K, int ldx, int ldw, int ldo, int inter, int w_static,
                    int* __restrict__ error_word, SbRope rp) {
-    constexpr bool GATED = MODE != SB_PLAIN;          // two row groups per strip
+    constexpr bool GATED = sb_two_groups(MODE);       // two row groups per strip
     constexpr int STRIPS = GATED ? 2 : 1;
     constexpr int GROUPS = STRIPS * NT;               // 8-row groups of a stage
     constexpr int ROWS = 8 * GROUPS;
@@ -187,7 +192,7 @@ smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT*
     constexpr int PER = SB_KC / 32 / SB_WARPS;
     auto load_x = [&](int strip, int ch, uint4 (&xv)[PER], uint4 (&xw)[PER]) {
         size_t plane = 0;
-        if (MODE == SB_PLAIN && rp.plane_rows > 0)
+        if (MODE == SB_PLANES)
             plane = (size_t)min(strip * 8 * NT / rp.plane_rows, rp.planes - 1) * rp.plane_stride;
 #pragma unroll
         for (int u = 0; u < PER; ++u) {
@@ -318,15 +323,15 @@ smallm_bulk_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, OutT*
                     const float r = fmaxf(__bfloat162float(__float2bfloat16_rn(y)), 0.f);
                     y = r * r;
                 }
-                if (MODE == SB_GATED) {
+                if (MODE == SB_GATED || MODE == SB_CLAMPED) {
                     // gate and up are rounded to bfloat16 first, as the unfused path stores them
                     const float gate = __bfloat162float(__float2bfloat16_rn(v[0]));
                     const float up = __bfloat162float(__float2bfloat16_rn(v[STRIPS - 1]));
                     // act 2: the tanh form of gelu, 0.5 g (1 + tanh z) = g / (1 + exp(-2 z))
                     const float z = rp.act == 2
                         ? 1.5957691216057308f * (gate + 0.044715f * gate * gate * gate) : gate;
-                    y = rp.act == 3 ? clamped_swish(gate, up, rp.limit, rp.alpha)
-                                    : gate / (1.f + expf(-z)) * up;
+                    y = MODE == SB_CLAMPED ? clamped_swish(gate, up, rp.limit, rp.alpha)
+                                           : gate / (1.f + expf(-z)) * up;
                 }
                 sb_store<OutT>(out + (size_t)m * ldo + n, y);
             }
@@ -341,7 +346,7 @@ static int launch_bulk_nt(const bf16* x, const bf16* W, OutT* out, int M, int n_
                           const SbRope& rp = SbRope{}) {
     static int resident = 0;   // CTAs of this variant that fit on the GPU at once
     auto kernel = smallm_bulk_kernel<MODE, M16, NT, OutT>;
-    constexpr int SMEM = sb_smem(MODE != SB_PLAIN, NT);
+    constexpr int SMEM = sb_smem(sb_two_groups(MODE), NT);
     if (resident == 0) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
         if (e != cudaSuccess) return (int)e;
@@ -382,19 +387,20 @@ static int pick_nt(int n_out, bool gated, bool m16) {
     return nt;
 }
 
-template <bool GATED, bool M16, typename OutT>
+template <int MODE, bool M16, typename OutT>
 static int launch_bulk(const bf16* x, const bf16* W, OutT* out, int M, int n_out, int K, int ldx, int ldw,
                        int ldo, int inter, int w_static, int* error_word, cudaStream_t s, int act = 0,
                        SbRope rp = SbRope{}) {
+    constexpr bool GATED = sb_two_groups(MODE);
     rp.act = act;
     int nt = pick_nt(n_out, GATED, M16);
-    while (rp.plane_rows > 0 && nt > 1 && rp.plane_rows % (8 * nt) != 0) nt /= 2;   // a strip has one plane
+    while (MODE == SB_PLANES && nt > 1 && rp.plane_rows % (8 * nt) != 0) nt /= 2;   // a strip has one plane
     switch (nt) {
         case 4:
             if constexpr (!GATED)
-                return launch_bulk_nt<GATED ? SB_GATED : SB_PLAIN, M16, 4, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
-        case 2: return launch_bulk_nt<GATED ? SB_GATED : SB_PLAIN, M16, 2, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
-        default: return launch_bulk_nt<GATED ? SB_GATED : SB_PLAIN, M16, 1, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
+                return launch_bulk_nt<MODE, M16, 4, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
+        case 2: return launch_bulk_nt<MODE, M16, 2, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
+        default: return launch_bulk_nt<MODE, M16, 1, OutT>(x, W, out, M, n_out, K, ldx, ldw, ldo, inter, w_static, error_word, s, rp);
     }
 }
 
@@ -419,20 +425,25 @@ MSTAR_API int mstar_gemm_smallm_bulk_bf16(const void* x, const void* W, void* ou
     const bf16* xp = (const bf16*)x;
     const bf16* wp = (const bf16*)W;
     if (gated) {
-        const int act = gated >= 2 ? gated : 0;
+        const int act = gated == 2 ? 2 : 0;
         SbRope rp{};
         rp.limit = limit;
         rp.alpha = alpha;
+        if (gated == 3) {
+            if (M > 8)
+                return launch_bulk<SB_CLAMPED, true, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, 0, rp);
+            return launch_bulk<SB_CLAMPED, false, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, 0, rp);
+        }
         if (M > 8)
-            return launch_bulk<true, true, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act, rp);
-        return launch_bulk<true, false, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act, rp);
+            return launch_bulk<SB_GATED, true, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act, rp);
+        return launch_bulk<SB_GATED, false, bf16>(xp, wp, (bf16*)out, M, N / 2, K, ldx, ldw, ldo, N / 2, w_static, error_word, s, act, rp);
     }
     if (out_dtype == MSTAR_F32) {
-        if (M > 8) return launch_bulk<false, true, float>(xp, wp, (float*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
-        return launch_bulk<false, false, float>(xp, wp, (float*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
+        if (M > 8) return launch_bulk<SB_PLAIN, true, float>(xp, wp, (float*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
+        return launch_bulk<SB_PLAIN, false, float>(xp, wp, (float*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
     }
-    if (M > 8) return launch_bulk<false, true, bf16>(xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
-    return launch_bulk<false, false, bf16>(xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
+    if (M > 8) return launch_bulk<SB_PLAIN, true, bf16>(xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
+    return launch_bulk<SB_PLAIN, false, bf16>(xp, wp, (bf16*)out, M, N, K, ldx, ldw, ldo, 0, w_static, error_word, s);
 }
 
 // out[M, N] = float products of the rows of W with several planes of x: features [p plane_rows, (p
@@ -451,9 +462,9 @@ MSTAR_API int mstar_gemm_smallm_bulk_planes(const void* x, const void* W, float*
     rp.planes = planes;
     rp.plane_stride = plane_stride;
     if (M > 8)
-        return launch_bulk<false, true, float>((const bf16*)x, (const bf16*)W, out, M, N, K, ldx, ldw, ldo, 0,
+        return launch_bulk<SB_PLANES, true, float>((const bf16*)x, (const bf16*)W, out, M, N, K, ldx, ldw, ldo, 0,
                                                w_static, error_word, (cudaStream_t)stream, 0, rp);
-    return launch_bulk<false, false, float>((const bf16*)x, (const bf16*)W, out, M, N, K, ldx, ldw, ldo, 0,
+    return launch_bulk<SB_PLANES, false, float>((const bf16*)x, (const bf16*)W, out, M, N, K, ldx, ldw, ldo, 0,
                                             w_static, error_word, (cudaStream_t)stream, 0, rp);
 }
 
@@ -467,9 +478,9 @@ MSTAR_API int mstar_gemm_smallm_bulk_relu2_bf16(const void* x, const void* W, vo
     if (((uintptr_t)x & 15) != 0 || ((uintptr_t)W & 15) != 0) return -1;
     cudaStream_t s = (cudaStream_t)stream;
     if (M > 8)
-        return launch_bulk<false, true, bf16>((const bf16*)x, (const bf16*)W, (bf16*)out, M, N, K, ldx, ldw,
+        return launch_bulk<SB_PLAIN, true, bf16>((const bf16*)x, (const bf16*)W, (bf16*)out, M, N, K, ldx, ldw,
                                               ldo, 0, w_static, error_word, s, 1);
-    return launch_bulk<false, false, bf16>((const bf16*)x, (const bf16*)W, (bf16*)out, M, N, K, ldx, ldw,
+    return launch_bulk<SB_PLAIN, false, bf16>((const bf16*)x, (const bf16*)W, (bf16*)out, M, N, K, ldx, ldw,
                                            ldo, 0, w_static, error_word, s, 1);
 }
 
