@@ -52,7 +52,9 @@ class PositionSpec:
 
 @dataclass(frozen=True)
 class NormSpec:
-    """kind "rmsnorm": ``x * rsqrt(mean(x^2) + eps) * (weight + weight_offset)``."""
+    """kind "rmsnorm": ``x * rsqrt(mean(x^2) + eps) * (weight + weight_offset)``.
+    kind "dynamic_tanh": ``tanh(alpha * x) * weight + bias``, alpha one learned number; no mean or
+    variance (``eps`` and ``weight_offset`` are not used)."""
 
     kind: str = "rmsnorm"
     size: int = 0
@@ -91,6 +93,11 @@ class AttentionSpec:
     p``, chunks counted from the sequence's start.  ``weights``: "softmax", or "sigmoid": the
     weight of a visible key is ``sigmoid(score)``, nothing is normalised over the keys.
     ``score_bias``: a learned number a head is added to the (scaled, capped) scores.
+    ``qk_norm_weight`` False: the norm a head has no weight (then it makes no difference whether
+    it stands before or after the rotation, which keeps a head's root mean square).
+    ``value_mix``: "first" hands this layer's values to later layers of the same step, "blend"
+    makes the values ``(1 - lam) v + lam v_first`` of the same token before they are cached, lam
+    a parameter (one number) and v_first the values of the run's "first" layer.
     """
 
     kind: str = "attention"
@@ -117,6 +124,8 @@ class AttentionSpec:
     chunk: Optional[int] = None
     weights: str = "softmax"
     score_bias: bool = False
+    qk_norm_weight: bool = True
+    value_mix: Optional[str] = None
 
     @property
     def value_dim(self) -> int:
@@ -129,7 +138,8 @@ class AttentionSpec:
                 and not self.bias and self.qk_norm_eps is None and self.conv_taps == 0
                 and not self.value_from_key and not self.head_gate and not self.feature_gate
                 and self.q_temp is None and self.softcap is None and self.sink is None
-                and self.chunk is None and self.weights == "softmax" and not self.score_bias)
+                and self.chunk is None and self.weights == "softmax" and not self.score_bias
+                and self.value_mix is None)
 
 
 @dataclass(frozen=True)
@@ -194,8 +204,8 @@ class ParallelMixerSpec:
 
 @dataclass(frozen=True)
 class GatedDeltaSpec:
-    """kind "gated_delta": a delta-rule matrix memory with a decay per head and key channel,
-    carried from token to token as per-request state.
+    """kind "gated_delta": a delta-rule matrix memory with a decay per head and key channel (or
+    one a head), carried from token to token as per-request state.
 
     ``q = W_q h`` and ``k = W_k h`` have ``num_kv_heads`` heads of ``qk_dim``, ``v = W_v h`` has
     ``num_heads`` heads of ``v_dim``; head h reads q/k head ``h // (num_heads / num_kv_heads)``.
@@ -206,7 +216,10 @@ class GatedDeltaSpec:
     row, ``u = beta (v - S^T k)``, ``S += k u^T``, ``o = S^T q``.  Each head's o is divided by
     its root mean square (``norm_eps``), scaled by a weight shared by the heads, gated by
     ``sigmoid(W_g2 W_g1 h)`` and projected back.  S (float) and the convolutions' last
-    ``conv - 1`` inputs are per-request state.
+    ``conv - 1`` inputs are per-request state.  ``head_decay``: one decay a head, ``exp(-exp(
+    A_log_h) * softplus(W_a h + dt_bias))`` (W_a has ``num_heads`` rows, ``decay_rank`` is not
+    used).  ``full_gate``: the gate is one product ``W_g h`` (``gate_rank`` is not used).
+    ``gate_activation``: "sigmoid" or "silu".
     """
 
     kind: str = "gated_delta"
@@ -221,6 +234,9 @@ class GatedDeltaSpec:
     norm_eps: float = 1e-6
     unit_eps: float = 1e-6
     shares_kv: bool = False
+    head_decay: bool = False
+    full_gate: bool = False
+    gate_activation: str = "sigmoid"
 
 
 @dataclass(frozen=True)
@@ -356,6 +372,10 @@ class RoutedExpertsSpec:
     -limit, limit)`` the hidden units are ``g sigmoid(swish_alpha g) (v + 1)``; the shared expert
     clamps at ``shared_limit``.  ``shared_gate``: the shared expert's output is multiplied by
     ``sigmoid(w_sg x)``, one number a token.
+    ``groups`` (count, keep): the experts form ``count`` equal groups of neighbours; a group
+    counts as its largest choice score (the correction included), and only experts of the best
+    ``keep`` groups can be chosen.  ``renorm_eps`` is added to the sum that the chosen scores are
+    divided by; ``weight_scale`` multiplies the weights at the end.
     """
 
     kind: str = "routed_experts"
@@ -375,16 +395,21 @@ class RoutedExpertsSpec:
     shared_limit: float = 0.0
     swish_alpha: float = 1.702
     shared_gate: bool = False
+    groups: Optional[tuple] = None
+    renorm_eps: float = 0.0
+    weight_scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class EmbeddingSpec:
-    """kind "table": the residual starts as ``table[token] * multiplier`` in float."""
+    """kind "table": the residual starts as ``table[token] * multiplier`` in float; ``norm``: a
+    norm spec that these rows pass first."""
 
     kind: str = "table"
     vocab_size: int = 0
     hidden_size: int = 0
     multiplier: float = 1.0
+    norm: Optional[object] = None
 
 
 @dataclass(frozen=True)

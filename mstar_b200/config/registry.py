@@ -113,3 +113,8 @@ def _register_builtin() -> None:
 
     if "Sokalorn" not in _ARCHITECTURES:
         register_architecture("Sokalorn", SokalornConfig, sokalorn_checkpoint_map)
+    from ..weights.famarax import famarax_checkpoint_map
+    from .famarax import FamaraxConfig
+
+    if "Famarax" not in _ARCHITECTURES:
+        register_architecture("Famarax", FamaraxConfig, famarax_checkpoint_map)

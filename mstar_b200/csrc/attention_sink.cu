@@ -13,7 +13,9 @@
 //             2i + 1; angle position * freq[i]); q goes to a dense [tokens, nq*hd] buffer, k
 //             and v into the token's cache page.  With `norm_whole` the root mean square is
 //             taken over all heads of q (and of k) at once and the weights have a number per
-//             feature of the whole projection.  With `temp_every` > 0 the query is multiplied
+//             feature of the whole projection; without weights the norm only divides.  With
+//             `v_first` the values become (1 - v_lam) v + v_lam v_first, another layer's values
+//             of the same token (float rows).  With `temp_every` > 0 the query is multiplied
 //             by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1).
 //   attend    the token whose key sits at cache position p sees keys j <= p with
 //             p - j < window or j < keep_first (window 0: every j <= p): the keys
@@ -43,6 +45,9 @@ struct PrepArgs {
     int norm_whole;             // 1: one root mean square over all q heads, one over all k heads
     float temp_coef;
     int temp_every;             // 0: no query temperature
+    const float* v_first;       // null, or float rows of v_first_stride with nkv*vd values each
+    int v_first_stride;
+    float v_lam;
 };
 
 // The convolved value of channel `col` (a column of q or k) of token t, the i-th of its
@@ -143,9 +148,12 @@ sink_prepare_kernel(const float* __restrict__ qkv, const W* __restrict__ bias,
             const int off = (a.nq + a.nkv) * a.hd + g * a.vd;
             A* dst = page_base + (size_t)a.nkv * a.page_size * a.hd +
                      ((size_t)g * a.page_size + slot) * a.vd;
+            const float* first = a.v_first == nullptr ? nullptr
+                                     : pdl_after(a.v_first, waited) + (size_t)t * a.v_first_stride + g * a.vd;
             for (int d = lane; d < a.vd; d += 32) {
                 float v = row[off + d];
                 if (bias != nullptr) v += to_float(bias[off + d]);
+                if (first != nullptr) v = fmaf(a.v_lam, first[d], (1.f - a.v_lam) * v);
                 dst[d] = from_float<A>(v);
             }
             continue;
@@ -176,12 +184,13 @@ sink_prepare_kernel(const float* __restrict__ qkv, const W* __restrict__ bias,
         const W* nw = is_q ? q_norm : k_norm;
         if (a.norm && a.norm_whole) {
             inv = is_q ? inv_whole_q : inv_whole_k;
-            nw += (size_t)(is_q ? h : h - a.nq) * a.hd;
+            if (nw != nullptr) nw += (size_t)(is_q ? h : h - a.nq) * a.hd;
         }
         const float mult = is_q ? q_mult : 1.f;
         __syncwarp();
         if (a.norm)
-            for (int d = lane; d < a.hd; d += 32) mine[d] = mine[d] * inv * to_float(nw[d]) * mult;
+            for (int d = lane; d < a.hd; d += 32)
+                mine[d] = mine[d] * inv * (nw != nullptr ? to_float(nw[d]) : 1.f) * mult;
         else if (mult != 1.f)
             for (int d = lane; d < a.hd; d += 32) mine[d] *= mult;
         __syncwarp();
@@ -216,8 +225,10 @@ MSTAR_API int mstar_sink_prepare(const float* qkv, const void* bias, const void*
                                  int row_stride, const void* conv_q, const void* conv_k, int taps,
                                  int v_from_k, const int* qo_indptr, const int* slots,
                                  const float* state, long long state_stride, int interleaved,
-                                 int norm_whole, float temp_coef, int temp_every, void* stream) {
+                                 int norm_whole, float temp_coef, int temp_every,
+                                 const float* v_first, int v_first_stride, float v_lam, void* stream) {
     if (tokens <= 0) return 0;
+    if (v_first != nullptr && (v_from_k || v_first_stride < nkv * vd)) return -1;
     if (norm_whole && taps > 0) return -1;
     if (hd <= 0 || vd <= 0 || rot < 0 || rot > hd || (rot & 1) || nq <= 0 || nkv <= 0) return -1;
     if (taps < 0 || (v_from_k && vd != hd)) return -1;
@@ -228,7 +239,8 @@ MSTAR_API int mstar_sink_prepare(const float* qkv, const void* bias, const void*
     const size_t smem = sizeof(float) * ((size_t)rot + (size_t)(threads / 32) * hd);
     if (smem > 48 * 1024) return -1;
     PrepArgs a{nq, nkv, hd, vd, rot, page_size, bt_stride, nq * hd, eps, norm, row_stride, taps,
-               v_from_k, state_stride, interleaved, norm_whole, temp_coef, temp_every};
+               v_from_k, state_stride, interleaved, norm_whole, temp_coef, temp_every,
+               v_first, v_first_stride, v_lam};
     cudaStream_t s = (cudaStream_t)stream;
     // a block takes 8 heads at a time: with fewer blocks than SMs, a token's heads go to
     // several blocks (each makes the token's sines and cosines for itself)

@@ -53,6 +53,36 @@ __device__ __forceinline__ void store8(bf16* p, const float (&v)[8]) {
     *reinterpret_cast<uint4*>(p) = raw;
 }
 
+// Four consecutive elements (the pointer must be aligned to 4 elements of T).
+__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void load4(const bf16* p, float (&v)[4]) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
+    uint2 raw;
+    *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
+    *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+// V = 4 or 1 of them.
+template <int V, typename T> __device__ __forceinline__ void load_v(const T* p, float (&v)[4]) {
+    if constexpr (V == 4) load4(p, v);
+    else v[0] = to_float(p[0]);
+}
+template <int V, typename T> __device__ __forceinline__ void store_v(T* p, const float (&v)[4]) {
+    if constexpr (V == 4) store4(p, v);
+    else p[0] = from_float<T>(v[0]);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -57,6 +57,138 @@ MSTAR_API int mstar_embed_rows(const void* table, int table_dtype, const int* id
     return launch_status();
 }
 
+// ------------------------------------------------- dynamic tanh
+// tanh(alpha v) * w + b, float: an elementwise "norm", so a row's columns are dealt out among
+// blocks (V columns a thread).  TABLE: v is the embedding row of a token (as above, times
+// `scale`) and out the float residual; else v = resid (+ delta, written back) and out has the
+// activation type.
+struct DynTanhArgs {
+    const void* table;          // TABLE: [vocab][hidden] in the weight type of the table
+    const int* ids;
+    const int* src;
+    const int* prev;
+    int vocab;
+    float scale;
+    float* resid;               // else: [rows][hidden]
+    const void* delta;          // null, or [rows][hidden] in the activation type
+    const void* weight;         // [hidden] each, weight type
+    const void* bias;
+    float alpha;
+    void* out;
+    int hidden;
+};
+
+template <typename A, typename W, int V>
+__global__ void __launch_bounds__(256) embed_tanh_kernel(DynTanhArgs a) {
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    const bool live = c < a.hidden;
+    float w[4], b[4];
+    if (live) {
+        load_v<V>(reinterpret_cast<const W*>(a.weight) + c, w);
+        load_v<V>(reinterpret_cast<const W*>(a.bias) + c, b);
+    }
+    const int* prev = pdl_after(a.prev, pdl_wait());     // sampled by the step before
+    if (!live) return;
+    const int t = blockIdx.x;
+    int id = a.ids[t];
+    if (a.src != nullptr) {
+        const int from = a.src[t];
+        if (from >= 0) id = prev[from];
+    }
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (id >= 0 && id < a.vocab)      // host validates ids; never read out of the table
+        load_v<V>(reinterpret_cast<const A*>(a.table) + (size_t)id * a.hidden + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = fmaf(tanhf(a.alpha * (v[e] * a.scale)), w[e], b[e]);
+    store_v<V>(reinterpret_cast<float*>(a.out) + (size_t)t * a.hidden + c, v);
+}
+
+template <typename A, typename W, int V>
+__global__ void __launch_bounds__(256) add_tanh_kernel(DynTanhArgs a) {
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    const bool live = c < a.hidden;
+    float w[4], b[4];
+    if (live) {
+        load_v<V>(reinterpret_cast<const W*>(a.weight) + c, w);
+        load_v<V>(reinterpret_cast<const W*>(a.bias) + c, b);
+    }
+    const unsigned long long waited = pdl_wait();
+    float* resid = pdl_after(a.resid, waited);
+    const A* delta = pdl_after(reinterpret_cast<const A*>(a.delta), waited);
+    if (!live) return;
+    const size_t at = (size_t)blockIdx.x * a.hidden + c;
+    float v[4];
+    load_v<V>(resid + at, v);
+    if (delta != nullptr) {
+        float d[4];
+        load_v<V>(delta + at, d);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] += d[e];
+        store_v<V>(resid + at, v);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = fmaf(tanhf(a.alpha * v[e]), w[e], b[e]);
+    store_v<V>(reinterpret_cast<A*>(a.out) + at, v);
+}
+
+static bool dyn_tanh_shape(const DynTanhArgs& a, int rows, dim3& grid, int& threads) {
+    bool vec = a.hidden % 4 == 0;
+    const void* ptrs[] = {a.table, a.resid, a.delta, a.weight, a.bias, a.out};
+    for (const void* p : ptrs) vec = vec && (uintptr_t)p % 16 == 0;
+    const int units = vec ? a.hidden / 4 : a.hidden;
+    threads = units >= 256 ? 256 : (units + 31) / 32 * 32;
+    grid = dim3(rows, (units + threads - 1) / threads);
+    return vec;
+}
+
+#define DYN_TANH_GO(KERNEL, A, W)                                                                \
+    do {                                                                                         \
+        if (vec) mstar_launch((KERNEL<A, W, 4>), grid, dim3(threads), 0, s, a);                  \
+        else mstar_launch((KERNEL<A, W, 1>), grid, dim3(threads), 0, s, a);                      \
+    } while (0)
+#define DYN_TANH_TYPES(KERNEL, first, second)                                                    \
+    do {                                                                                         \
+        if ((first) == MSTAR_F32) {                                                              \
+            if ((second) == MSTAR_F32) DYN_TANH_GO(KERNEL, float, float);                        \
+            else DYN_TANH_GO(KERNEL, float, bf16);                                               \
+        } else {                                                                                 \
+            if ((second) == MSTAR_F32) DYN_TANH_GO(KERNEL, bf16, float);                         \
+            else DYN_TANH_GO(KERNEL, bf16, bf16);                                                \
+        }                                                                                        \
+    } while (0)
+
+// Arguments as mstar_embed_rows, then the norm's.
+MSTAR_API int mstar_embed_tanh(const void* table, int table_dtype, const int* ids, const int* src,
+                               const int* prev, float* out, int num_tokens, int vocab, int hidden,
+                               float scale, const void* weight, const void* bias, int weight_dtype,
+                               float alpha, void* stream) {
+    if (num_tokens <= 0) return 0;
+    if ((src == nullptr) != (prev == nullptr) || hidden <= 0) return -1;
+    DynTanhArgs a{table, ids, src, prev, vocab, scale, nullptr, nullptr, weight, bias, alpha, out, hidden};
+    cudaStream_t s = (cudaStream_t)stream;
+    dim3 grid;
+    int threads;
+    const bool vec = dyn_tanh_shape(a, num_tokens, grid, threads);
+    DYN_TANH_TYPES(embed_tanh_kernel, table_dtype, weight_dtype);
+    return launch_status();
+}
+
+MSTAR_API int mstar_add_tanh(float* resid, const void* delta, const void* weight, const void* bias,
+                             int weight_dtype, float alpha, void* out, int act_dtype, int rows,
+                             int hidden, void* stream) {
+    if (rows <= 0) return 0;
+    if (hidden <= 0) return -1;
+    DynTanhArgs a{nullptr, nullptr, nullptr, nullptr, 0, 1.f, resid, delta, weight, bias, alpha, out, hidden};
+    cudaStream_t s = (cudaStream_t)stream;
+    dim3 grid;
+    int threads;
+    const bool vec = dyn_tanh_shape(a, rows, grid, threads);
+    DYN_TANH_TYPES(add_tanh_kernel, act_dtype, weight_dtype);
+    return launch_status();
+}
+#undef DYN_TANH_TYPES
+#undef DYN_TANH_GO
+
 // ------------------------------------------------- residual add + RMSNorm
 // resid (float, [rows, hidden]) is updated in place with resid + delta when delta
 // is given; out = resid * rsqrt(mean(resid^2) + eps) * (w + w_offset) in type A.

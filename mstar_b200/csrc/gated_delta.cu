@@ -7,12 +7,14 @@
 //            request's state slot, which holds the last taps - 1 projected rows) and SiLU;
 //            q and k heads to unit length (x / sqrt(sum x^2 + unit_eps)), q times D^-1/2;
 //            beta = sigmoid(b);  decay = exp(-exp(A_log_h) * softplus(a + dt_bias)) per head
-//            and key channel, a = the low-rank projection's output [H*D].
+//            and key channel, a = the low-rank projection's output [H*D].  With one decay a
+//            head (`head_decay`) a lies in the row behind b and the decays are [H].
 //   scan     per head, token after token:  S = decay * S (rows);  u = beta (v - S^T k);
 //            S += k u^T;  o = S^T q.  Computed as  r = (decay*S)^T k,  p = (decay*S)^T q,
 //            u = beta (v - r),  o = p + (q . k) u:  the chain from token to token holds one
 //            round of shuffles (r); the read-out's round runs beside the next token.
-//   finish   o / rms(o per head) * weight * sigmoid(gate), handed on in the activation type.
+//   finish   o / rms(o per head) * weight * sigmoid(gate) (or silu(gate)), handed on in the
+//            activation type.
 //
 // A slot is [(taps - 1) * (2 G D + H VD) convolution inputs | S^T as [H][VD][D]], float.
 // Everything here is float whatever the activation type.
@@ -24,8 +26,8 @@ struct DeltaPrepArgs {
     const float* proj;
     int row_stride;
     const void* conv_w;         // [2 G D + H VD][taps], weight type
-    const float* a_proj;        // [tokens][H*D]
-    const float* dt_bias;       // [H*D]
+    const float* a_proj;        // [tokens][H*D]; null: one decay a head, read from the row
+    const float* dt_bias;       // [H*D], or [H]
     const float* a_exp;         // [H]: exp(A_log)
     const int* token_req;
     const int* qo_indptr;
@@ -36,7 +38,7 @@ struct DeltaPrepArgs {
     float* k;                   // [tokens][G*D]
     float* v;                   // [tokens][H*VD]
     float* beta;                // [tokens][H]
-    float* decay;               // [tokens][H*D]
+    float* decay;               // [tokens][H*D], or [tokens][H]
     int H, G, D, VD, taps;
     float unit_eps;
 };
@@ -61,10 +63,53 @@ __device__ __forceinline__ float delta_conv_silu(const float* row, const float* 
     return y / (1.f + expf(-y));
 }
 
+// The same for four channels c .. c + 3 at once, by 16-byte accesses.
+template <typename W>
+__device__ __forceinline__ void delta_conv_silu4(const float* row, const float* slot, const W* cw,
+                                                 int c, int channels, int local,
+                                                 const DeltaPrepArgs& a, float (&y)[4]) {
+    const int keep = a.taps - 1;
+    y[0] = y[1] = y[2] = y[3] = 0.f;
+    if (a.taps == 4) {
+        float w[16], u[4][4];
+        if constexpr (sizeof(W) == 2) {
+            load8(cw + (size_t)c * 4, reinterpret_cast<float (&)[8]>(w[0]));
+            load8(cw + (size_t)c * 4 + 8, reinterpret_cast<float (&)[8]>(w[8]));
+        } else {
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                load4(cw + (size_t)c * 4 + 4 * i, reinterpret_cast<float (&)[4]>(w[4 * i]));
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int back = 3 - j;
+            load4(back <= local ? row - (ptrdiff_t)back * a.row_stride + c
+                                : slot + (size_t)(3 + local - back) * channels + c, u[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] = fmaf(w[4 * e + j], u[j][e], y[e]);
+    } else {
+        for (int j = 0; j < a.taps; ++j) {
+            const int back = keep - j;
+            float u[4];
+            load4(back <= local ? row - (ptrdiff_t)back * a.row_stride + c
+                                : slot + (size_t)(keep + local - back) * channels + c, u);
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                y[e] = fmaf(to_float(cw[(size_t)(c + e) * a.taps + j]), u[e], y[e]);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = y[e] / (1.f + expf(-y[e]));
+}
+
 // A block per token, or, with few tokens, several: a token's work comes in units that a warp
 // takes whole (a q head or a k head with its unit norm, the values of a head, the decays of a
-// head with its write strength), dealt out among the warps of gridDim.y blocks.
-template <typename W>
+// head with its write strength; with one decay a head, those of all heads), dealt out among the
+// warps of gridDim.y blocks.  VEC: heads, rows and buffers allow 16-byte accesses.
+template <typename W, bool VEC>
 __global__ void __launch_bounds__(256) delta_prepare_kernel(DeltaPrepArgs a) {
     extern __shared__ float ch[];             // [warps][D] a q or k head after its convolution
     const int t = blockIdx.x;
@@ -72,7 +117,7 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(DeltaPrepArgs a) {
     const W* cw = reinterpret_cast<const W*>(a.conv_w);
     const unsigned long long waited = pdl_wait();
     const float* proj = pdl_after(a.proj, waited);
-    const float* a_proj = pdl_after(a.a_proj, waited);
+    const float* a_proj = a.a_proj == nullptr ? nullptr : pdl_after(a.a_proj, waited);
     const float* state = pdl_after(a.state, waited);
     const int e = a.token_req[t];
     const int local = t - a.qo_indptr[e];
@@ -81,10 +126,24 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(DeltaPrepArgs a) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     float* mine = ch + (size_t)warp * a.D;
     const float q_scale = rsqrtf((float)a.D);
-    const int units = 2 * a.G + 2 * a.H;
+    const int units = 2 * a.G + a.H + (a_proj != nullptr ? a.H : 1);
     for (int u = blockIdx.y * nwarps + warp; u < units; u += nwarps * gridDim.y) {
         if (u < 2 * a.G) {                                // a q head, then the k heads
             float ss = 0.f;
+            if constexpr (VEC) {
+                if (a.D <= 128) {                         // a lane keeps its four in registers
+                    float y[4] = {0.f, 0.f, 0.f, 0.f};
+                    const int d = lane * 4;
+                    if (d < a.D) delta_conv_silu4(row, slot, cw, u * a.D + d, channels, local, a, y);
+                    ss = warp_sum(fmaf(y[0], y[0], y[1] * y[1]) + fmaf(y[2], y[2], y[3] * y[3]));
+                    const float inv = rsqrtf(ss + a.unit_eps) * (u < a.G ? q_scale : 1.f);
+                    float* dst = (u < a.G ? a.q : a.k) + (size_t)t * qk + (size_t)(u < a.G ? u : u - a.G) * a.D;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) y[e] *= inv;
+                    if (d < a.D) store4(dst + d, y);
+                    continue;
+                }
+            }
             for (int d = lane; d < a.D; d += 32) {
                 const float y = delta_conv_silu(row, slot, cw, u * a.D + d, channels, local, a);
                 mine[d] = y;
@@ -99,9 +158,23 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(DeltaPrepArgs a) {
             __syncwarp();
         } else if (u < 2 * a.G + a.H) {                   // the values of a head
             const int h = u - 2 * a.G;
-            for (int d = lane; d < a.VD; d += 32)
-                a.v[(size_t)t * vv + (size_t)h * a.VD + d] =
-                    delta_conv_silu(row, slot, cw, 2 * qk + h * a.VD + d, channels, local, a);
+            if constexpr (VEC) {
+                for (int d = lane * 4; d < a.VD; d += 128) {
+                    float y[4];
+                    delta_conv_silu4(row, slot, cw, 2 * qk + h * a.VD + d, channels, local, a, y);
+                    store4(a.v + (size_t)t * vv + (size_t)h * a.VD + d, y);
+                }
+            } else {
+                for (int d = lane; d < a.VD; d += 32)
+                    a.v[(size_t)t * vv + (size_t)h * a.VD + d] =
+                        delta_conv_silu(row, slot, cw, 2 * qk + h * a.VD + d, channels, local, a);
+            }
+        } else if (a_proj == nullptr) {                   // the decays and write strengths of all heads
+            for (int h = lane; h < a.H; h += 32) {
+                const float step = gd_softplus(row[channels + a.H + h] + a.dt_bias[h]);
+                a.decay[(size_t)t * a.H + h] = expf(-a.a_exp[h] * step);
+                a.beta[(size_t)t * a.H + h] = 1.f / (1.f + expf(-row[channels + h]));
+            }
         } else {                                          // the decays of a head, its write strength
             const int h = u - 2 * a.G - a.H;
             const float rate = a.a_exp[h];
@@ -125,7 +198,8 @@ MSTAR_API int mstar_delta_prepare(const float* proj, int row_stride, const void*
     if (tokens <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || VD <= 0 || taps < 1) return -1;
     const int channels = 2 * G * D + H * VD;
-    if (row_stride < channels + H) return -1;
+    const bool head_decay = a_proj == nullptr;
+    if (row_stride < channels + (head_decay ? 2 : 1) * H) return -1;
     if (taps > 1 && (!slots || !state)) return -1;
     const int threads = 256, warps = threads / 32;
     const size_t smem = sizeof(float) * (size_t)warps * D;
@@ -134,7 +208,7 @@ MSTAR_API int mstar_delta_prepare(const float* proj, int row_stride, const void*
                     state, state_stride, q, k, v, beta, decay, H, G, D, VD, taps, unit_eps};
     cudaStream_t s = (cudaStream_t)stream;
     // with fewer blocks than SMs a token's units go to several blocks
-    const int units = 2 * G + 2 * H;
+    const int units = 2 * G + H + (head_decay ? 1 : H);
     int parts = 1;
     if (tokens < device_sm_count()) {
         parts = (units + warps - 1) / warps;
@@ -143,22 +217,26 @@ MSTAR_API int mstar_delta_prepare(const float* proj, int row_stride, const void*
         if (parts < 1) parts = 1;
     }
     dim3 grid(tokens, parts);
-    static size_t configured_f = 0, configured_b = 0;
+    // 16-byte accesses: whole pieces per head, aligned rows, buffers and state
+    bool vec = D % 4 == 0 && VD % 4 == 0 && row_stride % 4 == 0 && state_stride % 4 == 0;
+    const void* ptrs[] = {proj, conv_w, state, q, k, v};
+    for (const void* p : ptrs) vec = vec && (uintptr_t)p % 16 == 0;
+#define GO1(W, VV)                                                                                \
+    do {                                                                                          \
+        static size_t configured = 0;                                                             \
+        if (smem > 48 * 1024 && smem > configured) {                                              \
+            cudaFuncSetAttribute(delta_prepare_kernel<W, VV>,                                     \
+                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+            configured = smem;                                                                    \
+        }                                                                                         \
+        mstar_launch((delta_prepare_kernel<W, VV>), grid, dim3(threads), smem, s, a);             \
+    } while (0)
     if (weight_dtype == MSTAR_F32) {
-        if (smem > 48 * 1024 && smem > configured_f) {
-            cudaFuncSetAttribute(delta_prepare_kernel<float>,
-                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-            configured_f = smem;
-        }
-        mstar_launch((delta_prepare_kernel<float>), grid, dim3(threads), smem, s, a);
+        if (vec) GO1(float, true); else GO1(float, false);
     } else {
-        if (smem > 48 * 1024 && smem > configured_b) {
-            cudaFuncSetAttribute(delta_prepare_kernel<bf16>,
-                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-            configured_b = smem;
-        }
-        mstar_launch((delta_prepare_kernel<bf16>), grid, dim3(threads), smem, s, a);
+        if (vec) GO1(bf16, true); else GO1(bf16, false);
     }
+#undef GO1
     return launch_status();
 }
 
@@ -200,11 +278,13 @@ __device__ __forceinline__ void gd_copy16(float* dst, const float* src) {
 // A warp that waits for its own shuffles has nothing else to issue, so a token's time is the
 // length of its instruction chain: the lanes of a column are as many as leave four rows a lane
 // (a whole warp a column from 128 rows on), R is the compiled number of rows a lane.
-// VEC: rows are whole 16-byte pieces (D a multiple of 4).
-template <int L, int R, bool VEC>
+// VEC: rows are whole 16-byte pieces (D a multiple of 4).  HD: one decay a head (`decay` is
+// [tokens][H] and travels with the write strength).
+template <int L, int R, bool VEC, bool HD>
 __global__ void __launch_bounds__(GD_THREADS) delta_scan_kernel(DeltaScanArgs a) {
-    extern __shared__ __align__(16) float stage[];     // [2][chunk][3 D + COLS + 4]
+    extern __shared__ __align__(16) float stage[];     // [2][chunk][NR D + COLS + 4]
     constexpr int COLS = GD_THREADS / L;
+    constexpr int NR = HD ? 2 : 3;                     // rows of a token: q, k (, decay)
     const int e = blockIdx.x, h = blockIdx.y;
     const int g = h / (a.H / a.G);
     const int lane = threadIdx.x % L;
@@ -214,7 +294,7 @@ __global__ void __launch_bounds__(GD_THREADS) delta_scan_kernel(DeltaScanArgs a)
     const bool live = col < a.VD;
     const int D = a.D;
     constexpr int DP = L * R;                          // rows as the lanes see them, zeros past D
-    const int per_tok = 3 * DP + COLS + 4;             // q, k, decay, values, beta (+ padding)
+    const int per_tok = NR * DP + COLS + 4;            // rows, values, beta, a head's decay (+ padding)
     const unsigned long long waited = pdl_wait();
     const float* q = pdl_after(a.q, waited);
     const float* k = pdl_after(a.k, waited);
@@ -233,7 +313,7 @@ __global__ void __launch_bounds__(GD_THREADS) delta_scan_kernel(DeltaScanArgs a)
         // copy i of the chunk is piece r of token j; both move on by fixed steps from copy to
         // copy, so the loop divides nothing
         const int unit = VEC ? 4 : 1;
-        const int per = 3 * (D / unit);                 // copies a token
+        const int per = NR * (D / unit);                // copies a token
         const int dj = GD_THREADS / per, dr = GD_THREADS % per;
         int j = threadIdx.x / per, r = threadIdx.x % per;
         for (; j < here; j += dj, r += dr) {
@@ -246,19 +326,21 @@ __global__ void __launch_bounds__(GD_THREADS) delta_scan_kernel(DeltaScanArgs a)
             float* dst = dst0 + (size_t)j * per_tok + which * DP + d;
             if constexpr (VEC) gd_copy16(dst, src); else gd_copy4(dst, src);
         }
-        for (int i = threadIdx.x; i < here * (ncols + 1); i += GD_THREADS) {
-            const int j = i / (ncols + 1), c = i - j * (ncols + 1);
+        constexpr int NS = HD ? 2 : 1;                  // numbers of a token: beta (, decay)
+        for (int i = threadIdx.x; i < here * (ncols + NS); i += GD_THREADS) {
+            const int j = i / (ncols + NS), c = i - j * (ncols + NS);
             const size_t tok = (size_t)(start + base + j);
-            float* dst = dst0 + (size_t)j * per_tok + 3 * DP;
+            float* dst = dst0 + (size_t)j * per_tok + NR * DP;
             if (c < ncols) gd_copy4(dst + c, v + tok * vv + (size_t)h * a.VD + col0 + c);
-            else gd_copy4(dst + COLS, beta + tok * a.H + h);
+            else if (c == ncols) gd_copy4(dst + COLS, beta + tok * a.H + h);
+            else gd_copy4(dst + COLS + 1, decay + tok * a.H + h);
         }
     };
 
     // rows past D read as zeros (q, k) whatever the chunk: no copy ever writes there
     if (DP > D) {
-        for (int i = threadIdx.x; i < 2 * a.chunk * 3 * (DP - D); i += GD_THREADS) {
-            const int j = i / (3 * (DP - D)), r = i - j * 3 * (DP - D);
+        for (int i = threadIdx.x; i < 2 * a.chunk * NR * (DP - D); i += GD_THREADS) {
+            const int j = i / (NR * (DP - D)), r = i - j * NR * (DP - D);
             stage[(size_t)j * per_tok + (r / (DP - D)) * DP + D + r % (DP - D)] = 0.f;
         }
     }
@@ -284,35 +366,32 @@ __global__ void __launch_bounds__(GD_THREADS) delta_scan_kernel(DeltaScanArgs a)
         const float* tokp = stage + (size_t)buf * a.chunk * per_tok;
         // the rows of the token after this one are read from shared memory while this one's
         // sums go round the lanes
-        float qn[R], kn[R], gn[R], vn, bn;
+        float qn[R], kn[R], gn[HD ? 1 : R], vn, bn;
+        auto next_rows = [&]() {
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-            qn[i] = tokp[lane + L * i];
-            kn[i] = tokp[DP + lane + L * i];
-            gn[i] = tokp[2 * DP + lane + L * i];
-        }
-        vn = tokp[3 * DP + mycol];
-        bn = tokp[3 * DP + COLS];
+            for (int i = 0; i < R; ++i) {
+                qn[i] = tokp[lane + L * i];
+                kn[i] = tokp[DP + lane + L * i];
+                if constexpr (!HD) gn[i] = tokp[2 * DP + lane + L * i];
+            }
+            if constexpr (HD) gn[0] = tokp[NR * DP + COLS + 1];
+            vn = tokp[NR * DP + mycol];
+            bn = tokp[NR * DP + COLS];
+        };
+        next_rows();
         for (int j = 0; j < here; ++j) {
-            float qr[R], kr[R], gr[R];
+            float qr[R], kr[R], gr[HD ? 1 : R];
 #pragma unroll
-            for (int i = 0; i < R; ++i) { qr[i] = qn[i]; kr[i] = kn[i]; gr[i] = gn[i]; }
+            for (int i = 0; i < R; ++i) { qr[i] = qn[i]; kr[i] = kn[i]; }
+#pragma unroll
+            for (int i = 0; i < (HD ? 1 : R); ++i) gr[i] = gn[i];
             const float vt = vn, bt = bn;
             tokp += per_tok;
-            if (j + 1 < here) {
-#pragma unroll
-                for (int i = 0; i < R; ++i) {
-                    qn[i] = tokp[lane + L * i];
-                    kn[i] = tokp[DP + lane + L * i];
-                    gn[i] = tokp[2 * DP + lane + L * i];
-                }
-                vn = tokp[3 * DP + mycol];
-                bn = tokp[3 * DP + COLS];
-            }
+            if (j + 1 < here) next_rows();
             float r4[4] = {0.f, 0.f, 0.f, 0.f}, p4[4] = {0.f, 0.f, 0.f, 0.f}, qkdot = 0.f;
 #pragma unroll
             for (int i = 0; i < R; ++i) {
-                s[i] *= gr[i];
+                s[i] *= gr[HD ? 0 : i];
                 r4[i & 3] = fmaf(kr[i], s[i], r4[i & 3]);
                 p4[i & 3] = fmaf(qr[i], s[i], p4[i & 3]);
                 qkdot = fmaf(qr[i], kr[i], qkdot);
@@ -353,7 +432,7 @@ MSTAR_API int mstar_delta_scan(const float* q, const float* k, const float* v, c
                                const float* decay, const int* qo_indptr, const int* slots,
                                float* state, long long state_stride, long long state_offset,
                                float* out, int entries, int max_q_len, int H, int G, int D, int VD,
-                               void* stream) {
+                               int head_decay, void* stream) {
     if (entries <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || VD <= 0 || D > 32 * GD_ROWS) return -1;
     if (H > 65535) return -1;
@@ -372,10 +451,10 @@ MSTAR_API int mstar_delta_scan(const float* q, const float* k, const float* v, c
     // (the staged rows are padded to L * R)
     // tokens staged at a time: 16, fewer where a token's rows are wide or the entries short
     int chunk = GD_CHUNK;
-    while (chunk > 1 && (chunk / 2 >= max_q_len ||
-                         (size_t)2 * chunk * (3 * L * R + cols + 4) * sizeof(float) > 64 * 1024))
+    const size_t per_tok = (size_t)(head_decay ? 2 : 3) * L * R + cols + 4;
+    while (chunk > 1 && (chunk / 2 >= max_q_len || 2 * chunk * per_tok * sizeof(float) > 64 * 1024))
         chunk /= 2;
-    const size_t smem = (size_t)2 * chunk * (3 * L * R + cols + 4) * sizeof(float);
+    const size_t smem = 2 * chunk * per_tok * sizeof(float);
     DeltaScanArgs a{q, k, v, beta, decay, qo_indptr, slots, state, state_stride, state_offset, out,
                     H, G, D, VD, chunk};
     cudaStream_t s = (cudaStream_t)stream;
@@ -383,20 +462,25 @@ MSTAR_API int mstar_delta_scan(const float* q, const float* k, const float* v, c
     if (grid.z > 65535) return -1;
     // 16-byte copies want whole pieces and aligned rows (the buffers are allocations of their own)
     const bool vec = D % 4 == 0 && (state_offset % 4) == 0 &&
-                     ((uintptr_t)q % 16 == 0) && ((uintptr_t)k % 16 == 0) && ((uintptr_t)decay % 16 == 0);
-#define GO1(LL, RR, VV)                                                                           \
+                     ((uintptr_t)q % 16 == 0) && ((uintptr_t)k % 16 == 0) &&
+                     (head_decay || (uintptr_t)decay % 16 == 0);
+#define GO1(LL, RR, VV, HH)                                                                           \
     do {                                                                                          \
         static size_t configured = 0;                                                             \
         if (smem > 48 * 1024 && smem > configured) {                                              \
-            cudaFuncSetAttribute(delta_scan_kernel<LL, RR, VV>,                                   \
+            cudaFuncSetAttribute(delta_scan_kernel<LL, RR, VV, HH>,                               \
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
             configured = smem;                                                                    \
         }                                                                                         \
-        mstar_launch((delta_scan_kernel<LL, RR, VV>), grid, dim3(GD_THREADS), smem, s, a);        \
+        mstar_launch((delta_scan_kernel<LL, RR, VV, HH>), grid, dim3(GD_THREADS), smem, s, a);    \
+    } while (0)
+#define GO2(LL, RR, VV)                                                                           \
+    do {                                                                                          \
+        if (head_decay) GO1(LL, RR, VV, true); else GO1(LL, RR, VV, false);                       \
     } while (0)
 #define GO(LL, RR)                                                                                \
     do {                                                                                          \
-        if (vec) GO1(LL, RR, true); else GO1(LL, RR, false);                                      \
+        if (vec) GO2(LL, RR, true); else GO2(LL, RR, false);                                      \
     } while (0)
     if (L == 4) GO(4, 4);
     else if (L == 8 && R == 4) GO(8, 4);
@@ -409,6 +493,7 @@ MSTAR_API int mstar_delta_scan(const float* q, const float* k, const float* v, c
     else if (R == 8) GO(32, 8);
     else GO(32, 16);
 #undef GO
+#undef GO2
 #undef GO1
     return launch_status();
 }
@@ -760,13 +845,444 @@ MSTAR_API int mstar_delta_scan_pieces(const float* q, const float* k, const floa
     return launch_status();
 }
 
+// ------------------------------------------------------------------ one decay a head, in pieces
+// With one decay g_t a head the decayed rows are the rows times a number, and everything inside a
+// piece of C tokens that does not depend on the state is a C x C matrix.  With P_t = g_1 .. g_t
+// (from the piece's first token), dec(t, j) = g_{j+1} .. g_t, the state S0 at the piece's start and
+//   L_tj = beta_t (k_t . k_j) dec(t, j)  (j < t),    B_tj = (q_t . k_j) dec(t, j)  (j <= t),
+// the delta rule of the piece is the triangular system (I + L) u = beta c, c_t = v_t - P_t k_t . S0:
+//   T = (I + L)^-1 diag(beta),   u = T c,   o_t = P_t q_t . S0 + (B T c)_t,
+//   S_C = P_C S0 + sum_j dec(C, j) k_j u_j.
+// A first kernel makes T, B T, P and dec(C, .) for all pieces and heads side by side (products of
+// decays only, never a quotient); the products of keys and queries among themselves are shared by
+// the heads of a group.  The scan reads the q and k rows as they are, several columns a warp, and
+// has no chain from token to token inside a piece.  All float.
+#define GH_WARPS 4
+#define GH_LD (GC_TOKENS + 4)       // floats between the rows of a C x C matrix in shared memory
+
+struct DeltaHeadArgs {
+    const float* q;
+    const float* k;
+    const float* v;
+    const float* beta;
+    const float* decay;         // [tokens][H]
+    const int* qo_indptr;
+    const int* slots;
+    float* T;                   // [H][tokens][C]
+    float* BT;                  // [H][tokens][C]
+    float* PS;                  // [H][tokens][2]: P_t, dec(C, t)
+    float* state;
+    long long state_stride;
+    long long state_offset;
+    float* out;
+    int H, G, D, VD, tokens;
+};
+
+// A block per (piece, entry, group of heads); thread (t, j) of 256 makes k_t . k_j and q_t . k_j,
+// then a warp a head: lane j the column j of T and of B T by forward substitution.
+__global__ void __launch_bounds__(256) delta_head_pieces_kernel(DeltaHeadArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int C = GC_TOKENS;
+    const int D = a.D, LD = D + 4;
+    float* ks = sm;                              // [C][LD]
+    float* qs = ks + C * LD;                     // [C][LD]
+    float* kk = qs + C * LD;                     // [C][GH_LD] k_t . k_j
+    float* qk = kk + C * GH_LD;                  // [C][GH_LD] q_t . k_j
+    float* per_warp = qk + C * GH_LD;            // [8 warps]{L, B [C][GH_LD], g, beta, prefix [C]}
+    const int piece = blockIdx.x, e = blockIdx.y, grp = blockIdx.z;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const unsigned long long waited = pdl_wait();
+    const float* q = pdl_after(a.q, waited);
+    const float* k = pdl_after(a.k, waited);
+    const float* beta = pdl_after(a.beta, waited);
+    const float* decay = pdl_after(a.decay, waited);
+    const int start = a.qo_indptr[e], n = a.qo_indptr[e + 1] - start;
+    const int base = piece * C;
+    if (base >= n) return;
+    const int here = min(C, n - base);
+    const int qkw = a.G * D;
+    for (int i = tid; i < C * (D / 4); i += 256) {
+        const int t = i / (D / 4), d = (i - t * (D / 4)) * 4;
+        float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv;
+        if (t < here) {
+            const size_t o = (size_t)(start + base + t) * qkw + (size_t)grp * D + d;
+            kv = *reinterpret_cast<const float4*>(k + o);
+            qv = *reinterpret_cast<const float4*>(q + o);
+        }
+        *reinterpret_cast<float4*>(ks + t * LD + d) = kv;
+        *reinterpret_cast<float4*>(qs + t * LD + d) = qv;
+    }
+    __syncthreads();
+    {
+        const int t = tid >> 4, j = tid & 15;
+        float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
+        for (int d = 0; d < D; d += 4) {
+            const float4 kt = *reinterpret_cast<const float4*>(ks + t * LD + d);
+            const float4 qt = *reinterpret_cast<const float4*>(qs + t * LD + d);
+            const float4 kj = *reinterpret_cast<const float4*>(ks + j * LD + d);
+            a0 = fmaf(kt.x, kj.x, a0); a1 = fmaf(kt.y, kj.y, a1);
+            b0 = fmaf(qt.x, kj.x, b0); b1 = fmaf(qt.y, kj.y, b1);
+            a0 = fmaf(kt.z, kj.z, a0); a1 = fmaf(kt.w, kj.w, a1);
+            b0 = fmaf(qt.z, kj.z, b0); b1 = fmaf(qt.w, kj.w, b1);
+        }
+        kk[t * GH_LD + j] = a0 + a1;
+        qk[t * GH_LD + j] = b0 + b1;
+    }
+    __syncthreads();
+    const int per = a.H / a.G;
+    float* L = per_warp + (size_t)warp * (2 * C * GH_LD + 2 * C);
+    float* B = L + C * GH_LD;
+    float* gs = B + C * GH_LD;
+    float* bs = gs + C;
+    for (int i = warp; i < per; i += 8) {
+        const int h = grp * per + i;
+        if (lane < C) {
+            const size_t o = (size_t)(start + base + lane) * a.H + h;
+            gs[lane] = lane < here ? decay[o] : 1.f;
+            bs[lane] = lane < here ? beta[o] : 0.f;
+        }
+        __syncwarp();
+        // lane (j, half): column j of L and B, dec(t, j) growing as t walks on; the lower half
+        // of the lanes writes L, the upper B
+        const int j = lane & 15;
+        float dec = 1.f;
+        for (int t = j; t < C; ++t) {
+            if (t > j) dec *= gs[t];
+            if (lane < C) { if (t > j) L[t * GH_LD + j] = bs[t] * kk[t * GH_LD + j] * dec; }
+            else B[t * GH_LD + j] = qk[t * GH_LD + j] * dec;
+        }
+        float P = 1.f;
+        for (int t = 0; t <= j; ++t) P *= gs[t];
+        __syncwarp();
+        if (lane < C) {
+            const size_t first = (size_t)h * a.tokens + start + base;
+            if (j < here) {
+                a.PS[(first + j) * 2] = P;
+                a.PS[(first + j) * 2 + 1] = dec;         // dec(C, j): a short piece's g are 1 past its end
+            }
+            float col[C];                                 // column j of (I + L)^-1
+#pragma unroll
+            for (int t = 0; t < C; ++t) {
+                float s = t == j ? 1.f : 0.f;
+#pragma unroll
+                for (int m = 0; m < t; ++m)
+                    if (m >= j) s = fmaf(-L[t * GH_LD + m], col[m], s);
+                col[t] = s;
+            }
+            const float bj = bs[j];
+#pragma unroll
+            for (int t = 0; t < C; ++t) {
+                float s = 0.f;
+#pragma unroll
+                for (int m = 0; m <= t; ++m)
+                    if (m >= j) s = fmaf(B[t * GH_LD + m], col[m], s);
+                if (t < here) {
+                    a.T[(first + t) * C + j] = t >= j ? col[t] * bj : 0.f;
+                    a.BT[(first + t) * C + j] = s * bj;
+                }
+            }
+        }
+        __syncwarp();
+    }
+}
+
+// Two floats multiplied and added at once.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 gh_fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 gh_pack(float lo, float hi) {
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float gh_both(f32x2 v) {
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+
+// A warp owns NC value columns of one head of one entry; a column's D = 32 R rows lie on the lanes,
+// R consecutive rows a lane.  Per piece: the columns go to shared memory; lane (t, half) takes
+// token t's products with all columns over one half of the rows (every key and query value it reads
+// meets NC columns); c goes round through shared memory, the lower lanes make u_t = (T c)_t, the
+// upper o_t; then the new columns.
+template <int R, int NC>
+__global__ void __launch_bounds__(GH_WARPS * 32) delta_head_scan_kernel(DeltaHeadArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int C = GC_TOKENS, D = 32 * R, LD = D + 4, COLS = GH_WARPS * NC;
+    constexpr int per_buf = 2 * C * LD + 2 * C * GH_LD + C * COLS + 2 * C;
+    static_assert(per_buf % 4 == 0, "the second buffer starts on a 16-byte boundary");
+    constexpr int per_warp = NC * D + NC * C + 2 * C * NC;
+    const int e = blockIdx.x, h = blockIdx.y;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int col0 = blockIdx.z * COLS;
+    float* mine = sm + 2 * per_buf + warp * per_warp;
+    float* cols = mine;                          // [NC][D] the columns at a piece's start
+    float* cs = cols + NC * D;                   // [NC][C]
+    float* us = cs + NC * C;                     // [C][NC][2] dec(C, t) u_t, each number twice
+    const unsigned long long waited = pdl_wait();
+    const float* q = pdl_after(a.q, waited);
+    const float* k = pdl_after(a.k, waited);
+    const float* v = pdl_after(a.v, waited);
+    const float* T = pdl_after((const float*)a.T, waited);
+    const float* BT = pdl_after((const float*)a.BT, waited);
+    const float* PS = pdl_after((const float*)a.PS, waited);
+    float* state = pdl_after(a.state, waited);
+    const int start = a.qo_indptr[e], n = a.qo_indptr[e + 1] - start;
+    if (n <= 0) return;
+    const int qkw = a.G * D, vv = a.H * a.VD, grp = h / (a.H / a.G);
+    const int ncols = min(COLS, a.VD - col0);
+
+    auto fetch = [&](int buf, int piece) {
+        const int base = piece * C;
+        const int here = min(C, n - base);
+        float* dst = sm + buf * per_buf;
+        const size_t first = (size_t)h * a.tokens + start + base;
+        for (int i = tid; i < here * (D / 4); i += GH_WARPS * 32) {
+            const int t = i / (D / 4), d = (i - t * (D / 4)) * 4;
+            const size_t o = (size_t)(start + base + t) * qkw + (size_t)grp * D + d;
+            gd_copy16(dst + t * LD + d, k + o);
+            gd_copy16(dst + C * LD + t * LD + d, q + o);
+        }
+        float* m = dst + 2 * C * LD;
+        for (int i = tid; i < here * (C / 4); i += GH_WARPS * 32) {
+            const int t = i / (C / 4), j = (i - t * (C / 4)) * 4;
+            gd_copy16(m + t * GH_LD + j, T + (first + t) * C + j);
+            gd_copy16(m + C * GH_LD + t * GH_LD + j, BT + (first + t) * C + j);
+        }
+        float* vs = m + 2 * C * GH_LD;
+        for (int i = tid; i < here * COLS; i += GH_WARPS * 32) {
+            const int t = i / COLS, c = i - t * COLS;
+            if (c < ncols)
+                gd_copy4(vs + t * COLS + c, v + (size_t)(start + base + t) * vv + (size_t)h * a.VD + col0 + c);
+        }
+        for (int i = tid; i < here * 2; i += GH_WARPS * 32) gd_copy4(vs + C * COLS + i, PS + first * 2 + i);
+    };
+
+    // what no copy writes (columns past the last, rows past a short piece) reads as finite numbers
+    for (int i = tid; i < 2 * per_buf; i += GH_WARPS * 32) sm[i] = 0.f;
+    __syncthreads();
+    const int pieces = (n + C - 1) / C;
+    fetch(0, 0);
+    cp_async_commit();
+    float* s_cols = state + (size_t)a.slots[e] * a.state_stride + a.state_offset +
+                    ((size_t)h * a.VD + col0 + warp * NC) * D;
+    float s[NC][R];
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        if (warp * NC + c < ncols) {
+            gc_load<R>(s_cols + (size_t)c * D + lane * R, s[c]);
+        } else {
+#pragma unroll
+            for (int i = 0; i < R; ++i) s[c][i] = 0.f;
+        }
+    }
+    const int t = lane & 15, half = lane >> 4;
+    for (int piece = 0; piece < pieces; ++piece) {
+        const int buf = piece & 1;
+        if (piece + 1 < pieces) fetch(buf ^ 1, piece + 1);
+        cp_async_commit();
+        cp_async_wait<1>();
+#pragma unroll
+        for (int c = 0; c < NC; ++c) gc_store<R>(cols + c * D + lane * R, s[c]);
+        __syncthreads();
+        const int here = min(C, n - piece * C);
+        const float* ks = sm + buf * per_buf;
+        const float* qs = ks + C * LD;
+        const float* ms = qs + C * LD;
+        const float* vs = ms + 2 * C * GH_LD;
+        const float* ps = vs + C * COLS;
+        f32x2 r2[NC], p2[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) r2[c] = p2[c] = 0ull;
+        {
+            const ulonglong2* kr = reinterpret_cast<const ulonglong2*>(ks + t * LD + half * (D / 2));
+            const ulonglong2* qr = reinterpret_cast<const ulonglong2*>(qs + t * LD + half * (D / 2));
+            const ulonglong2* sr = reinterpret_cast<const ulonglong2*>(cols + half * (D / 2));
+#pragma unroll
+            for (int i = 0; i < D / 8; ++i) {
+                const ulonglong2 k4 = kr[i], q4 = qr[i];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const ulonglong2 s4 = sr[c * (D / 4) + i];
+                    r2[c] = gh_fma2(k4.x, s4.x, r2[c]);
+                    p2[c] = gh_fma2(q4.x, s4.x, p2[c]);
+                    r2[c] = gh_fma2(k4.y, s4.y, r2[c]);
+                    p2[c] = gh_fma2(q4.y, s4.y, p2[c]);
+                }
+            }
+        }
+        const float P = ps[2 * t], dec = ps[2 * t + 1];
+        float o[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            float r = gh_both(r2[c]), p = gh_both(p2[c]);
+            r += __shfl_xor_sync(0xffffffffu, r, 16);
+            p += __shfl_xor_sync(0xffffffffu, p, 16);
+            o[c] = half ? P * p : 0.f;
+            // (a token past the piece has c = 0: its row and column of T and B T are not used)
+            if (half == 0) cs[c * C + t] = t < here ? vs[t * COLS + warp * NC + c] - P * r : 0.f;
+        }
+        __syncwarp();
+        {
+            const float4* row = reinterpret_cast<const float4*>(ms + half * C * GH_LD + t * GH_LD);
+            const float4* cv = reinterpret_cast<const float4*>(cs);
+#pragma unroll
+            for (int i = 0; i < C / 4; ++i) {
+                const float4 m4 = row[i];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const float4 c4 = cv[c * (C / 4) + i];
+                    o[c] = fmaf(m4.x, c4.x, o[c]);
+                    o[c] = fmaf(m4.y, c4.y, o[c]);
+                    o[c] = fmaf(m4.z, c4.z, o[c]);
+                    o[c] = fmaf(m4.w, c4.w, o[c]);
+                }
+            }
+        }
+        if (half == 0) {                         // o holds u_t here
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                const float u = t < here ? dec * o[c] : 0.f;
+                *reinterpret_cast<float2*>(us + (t * NC + c) * 2) = make_float2(u, u);
+            }
+        } else if (t < here) {
+            float* dst = a.out + (size_t)(start + piece * C + t) * vv + (size_t)h * a.VD + col0 + warp * NC;
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+                if (warp * NC + c < ncols) dst[c] = o[c];
+        }
+        __syncwarp();
+        const float PC = ps[2 * (here - 1)];
+        if constexpr (R >= 2) {
+            f32x2 s2[NC][R / 2];
+            const f32x2 pc2 = gh_pack(PC, PC);
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+#pragma unroll
+                for (int i = 0; i < R / 2; ++i)
+                    s2[c][i] = gh_fma2(gh_pack(s[c][2 * i], s[c][2 * i + 1]), pc2, 0ull);
+#pragma unroll 4
+            for (int j = 0; j < C; ++j) {
+                f32x2 kv[R / 2];
+                if constexpr (R == 2) {
+                    kv[0] = *reinterpret_cast<const f32x2*>(ks + j * LD + lane * R);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < R / 4; ++i) {
+                        const ulonglong2 k4 = reinterpret_cast<const ulonglong2*>(ks + j * LD + lane * R)[i];
+                        kv[2 * i] = k4.x;
+                        kv[2 * i + 1] = k4.y;
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < NC; c += 2) {
+                    const ulonglong2 u2 = *reinterpret_cast<const ulonglong2*>(us + (j * NC + c) * 2);
+#pragma unroll
+                    for (int i = 0; i < R / 2; ++i) {
+                        s2[c][i] = gh_fma2(kv[i], u2.x, s2[c][i]);
+                        s2[c + 1][i] = gh_fma2(kv[i], u2.y, s2[c + 1][i]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+#pragma unroll
+                for (int i = 0; i < R / 2; ++i)
+                    asm("mov.b64 {%0, %1}, %2;" : "=f"(s[c][2 * i]), "=f"(s[c][2 * i + 1]) : "l"(s2[c][i]));
+        } else {
+#pragma unroll
+            for (int c = 0; c < NC; ++c) s[c][0] *= PC;
+#pragma unroll 4
+            for (int j = 0; j < C; ++j) {
+                const float kv = ks[j * LD + lane];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) s[c][0] = fmaf(kv, us[(j * NC + c) * 2], s[c][0]);
+            }
+        }
+        __syncthreads();                       // the buffer is free for the piece after next
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+        if (warp * NC + c < ncols) gc_store<R>(s_cols + (size_t)c * D + lane * R, s[c]);
+}
+
+// The scan in pieces with one decay a head (`decay` [tokens][H]), for key sizes of 32, 64, 128 or
+// 256: `work` holds tokens * H * (2 * 16 + 2) floats.  Returns 0, a CUDA error code, or -1 when the
+// shape is refused.
+MSTAR_API int mstar_delta_scan_head_pieces(const float* q, const float* k, const float* v,
+                                           const float* beta, const float* decay,
+                                           const int* qo_indptr, const int* slots, float* state,
+                                           long long state_stride, long long state_offset, float* out,
+                                           float* work, int tokens, int entries, int max_q_len, int H,
+                                           int G, int D, int VD, void* stream) {
+    if (entries <= 0 || tokens <= 0) return 0;
+    if (H <= 0 || G <= 0 || H % G || VD <= 0) return -1;
+    if (D != 32 && D != 64 && D != 128 && D != 256) return -1;
+    if (H > 65535 || entries > 65535 || (state_offset % 4) != 0 || (state_stride % 4) != 0) return -1;
+    if ((uintptr_t)q % 16 || (uintptr_t)k % 16 || (uintptr_t)work % 16 || (uintptr_t)state % 16) return -1;
+    const int max_pieces = (max_q_len + GC_TOKENS - 1) / GC_TOKENS;
+    const size_t th = (size_t)tokens * H;
+    DeltaHeadArgs a{q, k, v, beta, decay, qo_indptr, slots, work, work + th * GC_TOKENS,
+                    work + 2 * th * GC_TOKENS, state, state_stride, state_offset, out, H, G, D, VD, tokens};
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem1 = (2 * (size_t)GC_TOKENS * (D + 4) + 2 * GC_TOKENS * GH_LD +
+                          8 * (2 * GC_TOKENS * GH_LD + 2 * GC_TOKENS)) * sizeof(float);
+    if (smem1 > 48 * 1024) {
+        static size_t configured = 0;
+        if (smem1 > configured) {
+            cudaFuncSetAttribute(delta_head_pieces_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                 (int)smem1);
+            configured = smem1;
+        }
+    }
+    mstar_launch(delta_head_pieces_kernel, dim3(max_pieces, entries, G), dim3(256), smem1, s, a);
+    int code = launch_status();
+    if (code != 0) return code;
+    // four columns a warp where that still gives half the SMs a block, else two
+    const int nc = (long long)entries * H * ((VD + 4 * GH_WARPS - 1) / (4 * GH_WARPS)) * 2 >=
+                           device_sm_count() ? 4 : 2;
+    const int cols = nc * GH_WARPS;
+    const size_t smem2 = ((size_t)2 * (2 * GC_TOKENS * (D + 4) + 2 * GC_TOKENS * GH_LD +
+                                       GC_TOKENS * cols + 2 * GC_TOKENS) +
+                          (size_t)GH_WARPS * (nc * D + nc * GC_TOKENS + 2 * GC_TOKENS * nc)) * sizeof(float);
+    dim3 grid(entries, H, (VD + cols - 1) / cols);
+    if (grid.z > 65535) return -1;
+#define GO1(RR, NN)                                                                               \
+    do {                                                                                          \
+        static size_t configured = 0;                                                             \
+        if (smem2 > 48 * 1024 && smem2 > configured) {                                            \
+            cudaFuncSetAttribute(delta_head_scan_kernel<RR, NN>,                                  \
+                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);        \
+            configured = smem2;                                                                   \
+        }                                                                                         \
+        mstar_launch((delta_head_scan_kernel<RR, NN>), grid, dim3(GH_WARPS * 32), smem2, s, a);   \
+    } while (0)
+#define GO(RR)                                                                                    \
+    do {                                                                                          \
+        if (nc == 4) GO1(RR, 4); else GO1(RR, 2);                                                 \
+    } while (0)
+    if (D == 32) GO(1);
+    else if (D == 64) GO(2);
+    else if (D == 128) GO(4);
+    else GO(8);
+#undef GO
+#undef GO1
+    return launch_status();
+}
+
 // ------------------------------------------------------------------ finish
-// out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * weight[:] * sigmoid(gate[t, h, :]) * scale; a
-// warp per (token, head).
-template <typename A>
-__global__ void delta_finish_kernel(const float* o, const A* gate, int gate_stride,
+// out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * weight[:] * act(gate[t, h, :]) * scale, act the
+// sigmoid or the SiLU; a warp per (token, head).  V: elements an access; a lane keeps up to four
+// accesses' worth of its head in registers.
+template <typename A, typename T, int V>
+__global__ void delta_finish_kernel(const float* o, const T* gate, int gate_stride,
                                     const float* __restrict__ weight, A* __restrict__ out,
-                                    int pairs, int heads, int vdim, float eps, float scale) {
+                                    int pairs, int heads, int vdim, float eps, float scale, int silu) {
     const unsigned long long waited = pdl_wait();
     o = pdl_after(o, waited);
     gate = pdl_after(gate, waited);
@@ -774,30 +1290,70 @@ __global__ void delta_finish_kernel(const float* o, const A* gate, int gate_stri
     if (pair >= pairs) return;
     const int t = pair / heads, h = pair - t * heads;
     const float* row = o + (size_t)pair * vdim;
+    const T* g = gate + (size_t)t * gate_stride + (size_t)h * vdim;
+    A* dst = out + (size_t)pair * vdim;
     float ss = 0.f;
+    if (vdim <= 128 * V) {
+        float v[4][4], z[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int j = (i * 32 + lane) * V;
+            if (j < vdim) {
+                load_v<V>(row + j, v[i]);
+                load_v<V>(g + j, z[i]);
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(v[i][e], v[i][e], ss);
+            }
+        }
+        const float inv = rsqrtf(warp_sum(ss) / (float)vdim + eps) * scale;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int j = (i * 32 + lane) * V;
+            if (j < vdim) {
+                float w[4];
+                load_v<V>(weight + j, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e)
+                    v[i][e] = v[i][e] * inv * w[e] / (1.f + expf(-z[i][e])) * (silu ? z[i][e] : 1.f);
+                store_v<V>(dst + j, v[i]);
+            }
+        }
+        return;
+    }
     for (int j = lane; j < vdim; j += 32) ss = fmaf(row[j], row[j], ss);
-    ss = warp_sum(ss);
-    const float inv = rsqrtf(ss / (float)vdim + eps) * scale;
-    const A* g = gate + (size_t)t * gate_stride + (size_t)h * vdim;
-    for (int j = lane; j < vdim; j += 32)
-        out[(size_t)pair * vdim + j] =
-            from_float<A>(row[j] * inv * weight[j] / (1.f + expf(-to_float(g[j]))));
+    const float inv = rsqrtf(warp_sum(ss) / (float)vdim + eps) * scale;
+    for (int j = lane; j < vdim; j += 32) {
+        const float z = to_float(g[j]);
+        dst[j] = from_float<A>(row[j] * inv * weight[j] / (1.f + expf(-z)) * (silu ? z : 1.f));
+    }
 }
 
+// gate_dtype: that of the activations, or float.
 MSTAR_API int mstar_delta_finish(const float* o, const void* gate, int gate_stride,
                                  const float* weight, void* out, int act_dtype, int tokens,
-                                 int heads, int vdim, float eps, float scale, void* stream) {
+                                 int heads, int vdim, float eps, float scale, int gate_dtype, int silu,
+                                 void* stream) {
     if (tokens <= 0) return 0;
+    if (gate_dtype != MSTAR_F32 && gate_dtype != act_dtype) return -1;
     const int pairs = tokens * heads, warps = 4;
     dim3 grid((pairs + warps - 1) / warps);
     cudaStream_t s = (cudaStream_t)stream;
-    if (act_dtype == MSTAR_F32)
-        mstar_launch((delta_finish_kernel<float>), grid, dim3(32 * warps), 0, s, o,
-                     (const float*)gate, gate_stride, weight, (float*)out, pairs, heads, vdim, eps,
-                     scale);
-    else
-        mstar_launch((delta_finish_kernel<bf16>), grid, dim3(32 * warps), 0, s, o,
-                     (const bf16*)gate, gate_stride, weight, (bf16*)out, pairs, heads, vdim, eps,
-                     scale);
+    const bool vec = vdim % 4 == 0 && gate_stride % 4 == 0 && (uintptr_t)o % 16 == 0 &&
+                     (uintptr_t)gate % 16 == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)out % 16 == 0;
+#define GO(A, T)                                                                                  \
+    do {                                                                                          \
+        if (vec)                                                                                  \
+            mstar_launch((delta_finish_kernel<A, T, 4>), grid, dim3(32 * warps), 0, s, o,         \
+                         (const T*)gate, gate_stride, weight, (A*)out, pairs, heads, vdim, eps,   \
+                         scale, silu);                                                            \
+        else                                                                                      \
+            mstar_launch((delta_finish_kernel<A, T, 1>), grid, dim3(32 * warps), 0, s, o,         \
+                         (const T*)gate, gate_stride, weight, (A*)out, pairs, heads, vdim, eps,   \
+                         scale, silu);                                                            \
+    } while (0)
+    if (act_dtype == MSTAR_F32) GO(float, float);
+    else if (gate_dtype == MSTAR_F32) GO(bf16, float);
+    else GO(bf16, bf16);
+#undef GO
     return launch_status();
 }

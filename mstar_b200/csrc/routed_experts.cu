@@ -5,6 +5,10 @@
 //   chosen  the `top` largest scores (the lower index wins a tie), weight w = s, or s divided
 //           by the sum of the chosen scores when `renormalize`
 //           With a `choice_bias` the largest of s + bias are chosen; the weights stay s.
+//           With `groups` > 0 the experts form that many equal groups of neighbours, a group
+//           counts as its largest choice score, and only experts of the best `keep` groups can
+//           be chosen.  `renorm_eps` is added to the sum the chosen scores are divided by;
+//           `weight_scale` multiplies the weights at the end.
 //   expert  y = W_down (silu(W_gate u) * (W_up u)),  u = w x (`scale_input`) or u = x with
 //           w multiplying y; without a gate (`gated` 0) y = W_down relu(W_up u)^2; `gated` 2
 //           takes the clamped swish of common.cuh (limit, alpha) for the SiLU and the product
@@ -28,6 +32,103 @@
 // comparison of (value, index), the lower index winning a tie.  Scores are monotone in the
 // logits, so the choice is made on the logits.
 #define RT_PER_LANE 32
+#define RT_MAX_GROUPS 1024
+
+// The largest (value, index) of a warp's lanes, the lower index winning a tie; an index of
+// 0x7fffffff is no candidate.
+__device__ __forceinline__ void rt_warp_best(float& bz, int& be) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float oz = __shfl_xor_sync(0xffffffffu, bz, o);
+        const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+        if (oe != 0x7fffffff && (be == 0x7fffffff || oz > bz || (oz == bz && oe < be))) {
+            bz = oz;
+            be = oe;
+        }
+    }
+}
+
+// The choice where it cannot be read off the logits alone: choice scores s + bias are made once
+// and kept in shared memory, and, with groups, the experts of all but the best `keep` groups are
+// closed.  A warp per token; the scores of a row lie at dynamic shared memory [warp][experts], the
+// groups' after all warps' scores ([warp][groups]).
+__global__ void route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ choice_bias,
+                                     int* __restrict__ chosen, float* __restrict__ weight, int tokens,
+                                     int experts, int top, int softmax, int renormalize, int ld,
+                                     int groups, int keep, float renorm_eps, float weight_scale) {
+    extern __shared__ float rt_sm[];
+    logits = pdl_after(logits, pdl_wait());
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const int t = blockIdx.x * nwarps + warp;
+    if (t >= tokens) return;
+    const float* z = logits + (size_t)t * ld;
+    float* choice = rt_sm + (size_t)warp * experts;
+    float* best = rt_sm + (size_t)nwarps * experts + (size_t)warp * groups;
+    float zmax = -INFINITY, denom = 1.f;
+    if (softmax) {
+        for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, z[e]);
+        zmax = warp_max(zmax);
+        denom = 0.f;
+        for (int e = lane; e < experts; e += 32) denom += expf(z[e] - zmax);
+        denom = warp_sum(denom);
+    }
+    auto score = [&](float v) { return softmax ? expf(v - zmax) / denom : 1.f / (1.f + expf(-v)); };
+    for (int e = lane; e < experts; e += 32)
+        choice[e] = score(z[e]) + (choice_bias != nullptr ? choice_bias[e] : 0.f);
+    __syncwarp();
+    const int per = groups > 0 ? experts / groups : experts;
+    // bit i: expert lane + 32 i cannot be chosen (any more)
+    unsigned closed = 0u;
+    if (groups > 0 && keep < groups) {
+        for (int g = lane; g < groups; g += 32) {
+            float m = choice[g * per];
+            for (int j = 1; j < per; ++j) m = fmaxf(m, choice[g * per + j]);
+            best[g] = m;
+        }
+        __syncwarp();
+        unsigned open_groups = 0u;              // bit i: group lane + 32 i is kept
+        for (int k = 0; k < keep; ++k) {
+            float bz = -INFINITY;
+            int be = 0x7fffffff;
+            for (int i = 0, g = lane; g < groups; ++i, g += 32)
+                if (!((open_groups >> i) & 1u) && (be == 0x7fffffff || best[g] > bz)) {
+                    bz = best[g];
+                    be = g;
+                }
+            rt_warp_best(bz, be);
+            if ((be & 31) == lane) open_groups |= 1u << (be >> 5);
+        }
+        // the mark of a kept group goes where every lane reads it
+        __syncwarp();
+        for (int i = 0, g = lane; g < groups; ++i, g += 32) best[g] = (open_groups >> i) & 1u ? 1.f : 0.f;
+        __syncwarp();
+        for (int i = 0, e = lane; e < experts; ++i, e += 32)
+            if (best[e / per] == 0.f) closed |= 1u << i;
+    }
+    float total = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float bz = -INFINITY;
+        int be = 0x7fffffff;
+        for (int i = 0, e = lane; e < experts; ++i, e += 32)
+            if (!((closed >> i) & 1u) && (be == 0x7fffffff || choice[e] > bz)) {
+                bz = choice[e];
+                be = e;
+            }
+        rt_warp_best(bz, be);
+        if ((be & 31) == lane) closed |= 1u << (be >> 5);
+        const float s = score(z[be]);
+        total += s;
+        if (lane == 0) {
+            chosen[(size_t)t * top + k] = be;
+            weight[(size_t)t * top + k] = s;
+        }
+    }
+    if (lane == 0) {
+        const float div = renormalize ? total + renorm_eps : 1.f;
+        for (int k = 0; k < top; ++k)
+            weight[(size_t)t * top + k] = weight[(size_t)t * top + k] / div * weight_scale;
+    }
+}
 
 __global__ void route_topk_kernel(const float* __restrict__ logits, const float* __restrict__ choice_bias,
                                   int* __restrict__ chosen,
@@ -89,10 +190,22 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, const float*
 
 MSTAR_API int mstar_route_topk(const float* logits, const float* choice_bias, int* chosen,
                                float* weight, int tokens, int experts, int top, int softmax,
-                               int renormalize, int ld, void* stream) {
+                               int renormalize, int ld, int groups, int keep, float renorm_eps,
+                               float weight_scale, void* stream) {
     if (tokens <= 0) return 0;
     if (ld < experts) return -1;
     if (experts <= 0 || top <= 0 || top > experts || experts > 32 * RT_PER_LANE) return -1;
+    if (groups > 0 && (groups > RT_MAX_GROUPS || experts % groups || keep <= 0 || keep > groups ||
+                       top > experts / groups * keep))
+        return -1;
+    if (groups > 0 || renorm_eps != 0.f || weight_scale != 1.f) {
+        // four warps' scores: at most 4 * (1,024 + 1,024) floats
+        const size_t smem = sizeof(float) * 4 * (size_t)(experts + (groups > 0 ? groups : 0));
+        mstar_launch(route_grouped_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream,
+                     logits, choice_bias, chosen, weight, tokens, experts, top, softmax, renormalize,
+                     ld, groups, keep, renorm_eps, weight_scale);
+        return launch_status();
+    }
     mstar_launch(route_topk_kernel, dim3((tokens + 3) / 4), dim3(128), 0, (cudaStream_t)stream,
                  logits, choice_bias, chosen, weight, tokens, experts, top, softmax, renormalize, ld);
     return launch_status();

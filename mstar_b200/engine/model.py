@@ -126,9 +126,7 @@ class Model:
         if want_rows is None or want_rows.numel() == 0:
             return torch.empty((0, self.vocab_size), dtype=torch.float32,
                                device=self.runtime.device)
-        rows = stream.gather(want_rows)
-        x = self.final_norm.norm_rows(rows)
-        return self.head.forward(x)
+        return self.head.forward(stream.gather_normed(want_rows, self.final_norm))
 
 
 def resolve_dtype(dtype) -> torch.dtype:

@@ -66,6 +66,50 @@ def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor | None 
     return out
 
 
+def _tanh_norm_args(norm, hidden: int) -> tuple:
+    """(weight pointer, bias pointer, their dtype code, alpha) of ``norm`` = (weight, bias, alpha)."""
+    weight, bias, alpha = norm
+    _need_cuda(weight, bias)
+    assert weight.numel() == hidden and bias.numel() == hidden and weight.dtype == bias.dtype
+    assert weight.is_contiguous() and bias.is_contiguous()
+    return weight.data_ptr(), bias.data_ptr(), _dt(weight), float(alpha)
+
+
+def embed_tanh(table: torch.Tensor, ids: torch.Tensor, norm, source=None, scale: float = 1.0):
+    """``embed_rows`` whose rows then pass a dynamic tanh, ``tanh(alpha * row) * weight + bias``
+    (``norm``: (weight, bias, alpha)); float."""
+    _need_cuda(table, ids)
+    assert ids.dtype == torch.int32 and table.dim() == 2 and table.is_contiguous()
+    n, (vocab, hidden) = ids.numel(), table.shape
+    out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
+    src = prev = None
+    if source is not None:
+        src, prev = source
+        _need_cuda(src, prev)
+        assert src.dtype == torch.int32 and prev.dtype == torch.int32 and src.numel() == n
+    w, b, wd, alpha = _tanh_norm_args(norm, hidden)
+    check(lib.get("elementwise").mstar_embed_tanh(
+        table.data_ptr(), _dt(table), ids.data_ptr(), _ptr(src), _ptr(prev), out.data_ptr(), n,
+        vocab, hidden, float(scale), w, b, wd, alpha, _stream()), "embed_tanh")
+    return out
+
+
+def add_tanh(resid: torch.Tensor, delta, norm, out_dtype: torch.dtype):
+    """resid += delta (if given), in place in float; returns ``tanh(alpha * resid) * weight + bias``
+    in ``out_dtype`` (``norm``: (weight, bias, alpha))."""
+    _need_cuda(resid, delta)
+    assert resid.dtype == torch.float32 and resid.dim() == 2 and resid.is_contiguous()
+    rows, hidden = resid.shape
+    if delta is not None:
+        assert delta.shape == resid.shape and delta.dtype == out_dtype and delta.is_contiguous()
+    out = torch.empty((rows, hidden), dtype=out_dtype, device=resid.device)
+    w, b, wd, alpha = _tanh_norm_args(norm, hidden)
+    check(lib.get("elementwise").mstar_add_tanh(
+        resid.data_ptr(), _ptr(delta), w, b, wd, alpha, out.data_ptr(), _dt(out), rows, hidden,
+        _stream()), "add_tanh")
+    return out
+
+
 def scale_softcap(x: torch.Tensor, scale: float = 1.0, cap: float | None = None):
     """In place on float ``x``: x *= scale, then x = cap * tanh(x / cap) if ``cap``."""
     _need_cuda(x)
@@ -1150,10 +1194,13 @@ def linear_per_head(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | N
 
 # ------------------------------------------------------------------ routed experts
 def route_topk(logits: torch.Tensor, top: int, softmax: bool = False, renormalize: bool = False,
-               choice_bias=None):
+               choice_bias=None, groups=None, renorm_eps: float = 0.0, weight_scale: float = 1.0):
     """(chosen int32 [tokens, top], weight float [tokens, top]) from float router logits (a
     column view of a wider product will do).
-    ``choice_bias``: float [experts] added to the scores for the choice only."""
+    ``choice_bias``: float [experts] added to the scores for the choice only.  ``groups``: (count,
+    keep) leaves only the experts of the ``keep`` groups with the largest choice score in them (of
+    ``count`` equal groups of neighbours).  ``renorm_eps`` is added to the sum that chosen scores
+    are divided by; the weights are multiplied by ``weight_scale``."""
     _need_cuda(logits, choice_bias)
     assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.stride(1) == 1
     tokens, experts = logits.shape
@@ -1163,9 +1210,11 @@ def route_topk(logits: torch.Tensor, top: int, softmax: bool = False, renormaliz
     weight = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     code = lib.get("routed_experts").mstar_route_topk(
         logits.data_ptr(), _ptr(choice_bias), chosen.data_ptr(), weight.data_ptr(), tokens, experts, top,
-        int(softmax), int(renormalize), logits.stride(0), _stream())
+        int(softmax), int(renormalize), logits.stride(0), *(groups or (0, 0)), float(renorm_eps),
+        float(weight_scale), _stream())
     if code == -1:
-        raise KernelError(f"cannot choose {top} of {experts} experts")
+        raise KernelError(f"cannot choose {top} of {experts} experts"
+                          + (f" in the best {groups[1]} of {groups[0]} groups" if groups else ""))
     check(code, "route_topk")
     return chosen, weight
 
@@ -1289,7 +1338,7 @@ def sink_prepare(qkv: torch.Tensor, bias, q_norm, k_norm, freq, positions, cache
                  head_dim: int, v_dim: int, rot: int, page_size: int, eps: float,
                  out_dtype: torch.dtype, conv=None, value_from_key: bool = False,
                  interleaved: bool = False, norm_whole: bool = False,
-                 q_temp=None) -> torch.Tensor:
+                 q_temp=None, norm: bool | None = None, first_values=None) -> torch.Tensor:
     """From the float fused projection ``qkv`` [tokens, (heads + kv_heads) * head_dim +
     kv_heads * v_dim (+ columns this kernel does not read)]: add ``bias``, norm every query
     and key head (``q_norm`` / ``k_norm`` weights of ``head_dim``, or None for no norm), rotate
@@ -1305,7 +1354,16 @@ def sink_prepare(qkv: torch.Tensor, bias, q_norm, k_norm, freq, positions, cache
     ``norm_whole``: one root mean square over all query heads and one over all key heads;
     ``q_norm`` / ``k_norm`` then have ``heads * head_dim`` / ``kv_heads * head_dim`` numbers.
     ``q_temp``: (coef, every) multiplies the query of the token at position p by ``1 + coef
-    * ln(floor((p + 1) / every) + 1)``."""
+    * ln(floor((p + 1) / every) + 1)``.  ``norm`` True without norm weights: the heads are
+    divided by their root mean square and nothing else.  ``first_values``: (float [tokens, kv_heads
+    * v_dim] rows, lam): the values become ``(1 - lam) v + lam * rows``."""
+    norm = q_norm is not None if norm is None else bool(norm)
+    mix_rows, lam = first_values if first_values is not None else (None, 0.0)
+    if mix_rows is not None:
+        _need_cuda(mix_rows)
+        assert mix_rows.dtype == torch.float32 and mix_rows.stride(1) == 1 and not value_from_key
+        assert tuple(mix_rows.shape) == (qkv.shape[0], num_kv_heads * v_dim)
+    assert norm or q_norm is None
     _need_cuda(qkv, bias, q_norm, k_norm, freq, positions, cache_pos, token_req, block_table,
                kv_cache)
     if q_norm is not None:
@@ -1345,10 +1403,11 @@ def sink_prepare(qkv: torch.Tensor, bias, q_norm, k_norm, freq, positions, cache
         qkv.data_ptr(), _ptr(bias), _ptr(q_norm), _ptr(k_norm), wd, _ptr(freq),
         positions.data_ptr(), cache_pos.data_ptr(), token_req.data_ptr(), block_table.data_ptr(),
         block_table.stride(0), q.data_ptr(), kv_cache.data_ptr(), _DT[out_dtype], tokens, num_heads,
-        num_kv_heads, head_dim, v_dim, rot, page_size, float(eps), int(q_norm is not None),
+        num_kv_heads, head_dim, v_dim, rot, page_size, float(eps), int(norm),
         qkv.stride(0), _ptr(wq), _ptr(wk), taps, int(value_from_key), _ptr(qo), _ptr(slots),
         _ptr(state) if taps > 1 else 0, state.stride(0) if taps > 1 else 0, int(interleaved),
-        int(norm_whole and q_norm is not None), temp_coef, temp_every, _stream())
+        int(norm_whole and norm), temp_coef, temp_every, _ptr(mix_rows),
+        mix_rows.stride(0) if mix_rows is not None else 0, float(lam), _stream())
     if code == -1:
         raise KernelError(f"attention input kernel refuses head_dim={head_dim}, v_dim={v_dim}, "
                           f"rot={rot}, taps={taps}")
@@ -1580,7 +1639,8 @@ def selective_scan(xc: torch.Tensor, xz: torch.Tensor, proj: torch.Tensor, w_dt,
 # ------------------------------------------------------------------ hyper-connections
 def hyper_step(x: torch.Tensor, *, init=None, y=None, y2=None, y_scales=(1.0, 1.0), y_bias=None,
                mix=None, out=None, read=None, norm_weight=None, eps: float = 0.0,
-               out_dtype: torch.dtype | None = None, rows=None):
+               out_dtype: torch.dtype | None = None, rows=None, tanh_norm=None,
+               x_static: bool = False):
     """What lies between two sublayers of a residual kept as copies ``x`` [tokens, S, width]
     (float, updated in place).
 
@@ -1589,7 +1649,12 @@ def hyper_step(x: torch.Tensor, *, init=None, y=None, y2=None, y_scales=(1.0, 1.
     y``.  With ``init`` [tokens, width] the old copies are all that row.  Then either ``read``
     (float [S]) with ``norm_weight``: returns ``rmsnorm(sum_s read[s] x_s) * norm_weight`` in
     ``out_dtype``; or ``rows`` (int32 indices): returns float ``sum_s x_s`` of those tokens
-    without writing the copies back."""
+    without writing the copies back.
+
+    ``tanh_norm``: (weight, bias, alpha) of a dynamic tanh in place of the RMS norm; the summed
+    rows pass it too (and come back in ``out_dtype``).  ``x_static`` promises that the kernel before
+    this one on the stream did not write ``x``: that norm's kernel then reads it while the other
+    drains."""
     _need_cuda(x, init, y, y2, y_bias, mix, out, read, norm_weight, rows)
     assert x.dtype == torch.float32 and x.dim() == 3 and x.is_contiguous()
     tokens, streams, width = x.shape
@@ -1612,6 +1677,23 @@ def hyper_step(x: torch.Tensor, *, init=None, y=None, y2=None, y_scales=(1.0, 1.
     for w in (y_bias, norm_weight):
         assert w is None or (_dt(w) == wd and w.is_contiguous() and w.numel() == width)
     normed = sums = None
+    if tanh_norm is not None:
+        assert out_dtype is not None
+        assert read is None or (read.dtype == torch.float32 and read.numel() == streams)
+        assert rows is None or (rows.dtype == torch.int32 and rows.is_contiguous())
+        blocks = tokens if rows is None else rows.numel()
+        w, b, td, alpha = _tanh_norm_args(tanh_norm, width)
+        assert y_bias is None or td == wd
+        normed = torch.empty((blocks, width), dtype=out_dtype, device=x.device)
+        code = lib.get("hyper").mstar_hyper_step_tanh(
+            x.data_ptr(), _ptr(init), _ptr(y), _ptr(y2), _ptr(y_bias), float(y_scales[0]),
+            float(y_scales[1]), mix.data_ptr(), out.data_ptr(), _ptr(read), w, b, alpha,
+            normed.data_ptr(), _ptr(rows), blocks, streams, width, int(x_static), _DT[out_dtype], td,
+            _stream())
+        if code == -1:
+            raise KernelError(f"hyper-connection kernel refuses streams={streams}, width={width}")
+        check(code, "hyper_step_tanh")
+        return normed
     if read is not None:
         assert read.dtype == torch.float32 and read.numel() == streams
         assert norm_weight is not None and out_dtype is not None
@@ -1671,7 +1753,8 @@ def gated_delta_state_size(heads: int, kv_heads: int, dim: int, vdim: int, taps:
 def delta_prepare(proj: torch.Tensor, conv_w: torch.Tensor, a_proj: torch.Tensor, dt_bias, a_exp,
                   token_req, qo_indptr, slots, state: torch.Tensor, heads: int, kv_heads: int,
                   dim: int, vdim: int, taps: int, unit_eps: float):
-    """From the float fused projection ``proj`` [tokens, q | k | v | b | ...]: convolution and
+    """From the float fused projection ``proj`` [tokens, q | k | v | b | a | ...] (``a`` only with
+    ``a_proj`` None: one decay a head; the decays are then [tokens, heads]): convolution and
     SiLU on the q, k and v channels (``conv_w`` [channels, taps]; rows before a portion from
     ``state``), unit q (times ``dim ** -0.5``) and k per head, ``beta = sigmoid(b)``, and the
     decays ``exp(-a_exp[h] * softplus(a_proj + dt_bias))``.  Returns float (q, k, v, beta,
@@ -1681,9 +1764,13 @@ def delta_prepare(proj: torch.Tensor, conv_w: torch.Tensor, a_proj: torch.Tensor
     qk, vv = kv_heads * dim, heads * vdim
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= 2 * qk + vv + heads
     assert tuple(conv_w.shape) == (2 * qk + vv, taps) and conv_w.is_contiguous()
-    assert a_proj.dtype == torch.float32 and a_proj.is_contiguous()
-    assert tuple(a_proj.shape) == (tokens, heads * dim)
-    assert dt_bias.dtype == torch.float32 and dt_bias.numel() == heads * dim
+    decays = heads if a_proj is None else heads * dim
+    if a_proj is None:
+        assert proj.shape[1] >= 2 * qk + vv + 2 * heads
+    else:
+        assert a_proj.dtype == torch.float32 and a_proj.is_contiguous()
+        assert tuple(a_proj.shape) == (tokens, decays)
+    assert dt_bias.dtype == torch.float32 and dt_bias.numel() == decays
     assert a_exp.dtype == torch.float32 and a_exp.numel() == heads
     assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
     assert state.shape[1] >= gated_delta_state_size(heads, kv_heads, dim, vdim, taps)
@@ -1692,9 +1779,9 @@ def delta_prepare(proj: torch.Tensor, conv_w: torch.Tensor, a_proj: torch.Tensor
     k = torch.empty((tokens, qk), dtype=torch.float32, device=dev)
     v = torch.empty((tokens, vv), dtype=torch.float32, device=dev)
     beta = torch.empty((tokens, heads), dtype=torch.float32, device=dev)
-    decay = torch.empty((tokens, heads * dim), dtype=torch.float32, device=dev)
+    decay = torch.empty((tokens, decays), dtype=torch.float32, device=dev)
     code = lib.get("gated_delta").mstar_delta_prepare(
-        proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), _dt(conv_w), a_proj.data_ptr(),
+        proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), _dt(conv_w), _ptr(a_proj),
         dt_bias.data_ptr(), a_exp.data_ptr(), token_req.data_ptr(), qo_indptr.data_ptr(),
         slots.data_ptr(), state.data_ptr(), state.stride(0), q.data_ptr(), k.data_ptr(),
         v.data_ptr(), beta.data_ptr(), decay.data_ptr(), tokens, heads, kv_heads, dim, vdim, taps,
@@ -1722,12 +1809,15 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
     scanned in pieces of 16 tokens: what does not depend on the state (decayed keys and
     queries, the keys' products among themselves) is made for all pieces side by side, and
     the chain from token to token shrinks to a scalar a token (MSTAR_DELTA_PIECES=0: never;
-    1: always)."""
+    1: always).  ``decay`` [tokens, heads] is one decay a head: the chain inside a piece then
+    becomes a small triangular matrix made ahead."""
     _need_cuda(q, k, v, beta, decay, qo_indptr, slots, state)
     for t in (q, k, v, beta, decay):
         assert t.dtype == torch.float32 and t.is_contiguous()
     assert state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
     tokens = q.shape[0]
+    head_decay = tuple(decay.shape) == (tokens, heads) and dim > 1
+    assert head_decay or tuple(decay.shape) == (tokens, heads * dim)
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=q.device)
     offset = (taps - 1) * (2 * kv_heads * dim + heads * vdim)
     longest = int(min(max_q_len, tokens))
@@ -1736,6 +1826,20 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
     if (pieces and dim in DELTA_PIECES_DIMS and tokens > 0 and offset % 4 == 0
             and state.stride(0) % 4 == 0):
         max_pieces = -(-longest // DELTA_PIECE)
+        if head_decay:
+            work = torch.empty(tokens * heads * (2 * DELTA_PIECE + 2), dtype=torch.float32,
+                               device=q.device)
+            code = lib.get("gated_delta").mstar_delta_scan_head_pieces(
+                q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), decay.data_ptr(),
+                qo_indptr.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0), offset,
+                out.data_ptr(), work.data_ptr(), tokens, entries, longest, heads, kv_heads, dim,
+                vdim, _stream())
+            if code == -1:
+                raise KernelError(f"delta-rule scan in pieces refuses heads={heads}, "
+                                  f"kv_heads={kv_heads}, dim={dim}")
+            check(code, "delta_scan_head_pieces")
+            lib.add_launches(1)
+            return out
         floats = (3 * tokens * heads * dim + entries * max_pieces * heads * dim
                   + 2 * tokens * heads * DELTA_PIECE)
         work = torch.empty(floats, dtype=torch.float32, device=q.device)
@@ -1754,7 +1858,7 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
         q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), decay.data_ptr(),
         qo_indptr.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0), offset,
         out.data_ptr(), entries, int(min(max_q_len, 1 << 30)), heads, kv_heads, dim, vdim,
-        _stream())
+        int(head_decay), _stream())
     if code == -1:
         raise KernelError(f"delta-rule scan refuses heads={heads}, kv_heads={kv_heads}, dim={dim} "
                           "(dim at most 512)")
@@ -1763,18 +1867,22 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
 
 
 def delta_finish(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, heads: int, vdim: int,
-                 eps: float, out_dtype: torch.dtype, scale: float = 1.0) -> torch.Tensor:
-    """o / rms(o per head) * weight * sigmoid(gate) * scale: float ``o`` [tokens, heads * vdim],
-    ``gate`` of the same shape in ``out_dtype``, float ``weight`` [vdim] shared by the heads."""
+                 eps: float, out_dtype: torch.dtype, scale: float = 1.0,
+                 gate_activation: str = "sigmoid") -> torch.Tensor:
+    """o / rms(o per head) * weight * sigmoid(gate) * scale (``gate_activation`` "silu": gate *
+    sigmoid(gate)): float ``o`` [tokens, heads * vdim], ``gate`` of the same shape in ``out_dtype``
+    or float (a column view of a wider product will do), float ``weight`` [vdim] shared by the
+    heads."""
+    assert gate_activation in ("sigmoid", "silu")
     _need_cuda(o, gate, weight)
     assert o.dtype == torch.float32 and o.is_contiguous()
     assert weight.dtype == torch.float32 and weight.numel() == vdim
-    assert gate.dtype == out_dtype and gate.stride(1) == 1 and gate.shape == o.shape
+    assert gate.dtype in (out_dtype, torch.float32) and gate.stride(1) == 1 and gate.shape == o.shape
     out = torch.empty(o.shape, dtype=out_dtype, device=o.device)
     check(lib.get("gated_delta").mstar_delta_finish(
         o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), out.data_ptr(),
-        _DT[out_dtype], o.shape[0], heads, vdim, float(eps), float(scale), _stream()),
-        "delta_finish")
+        _DT[out_dtype], o.shape[0], heads, vdim, float(eps), float(scale), _dt(gate),
+        int(gate_activation == "silu"), _stream()), "delta_finish")
     return out
 
 

@@ -21,6 +21,8 @@ _SIGNATURES = {
     "elementwise": {
         "mstar_embed_rows": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp],
         "mstar_scale_softcap": [_vp, _ll, _f, _f, _vp],
+        "mstar_embed_tanh": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp, _vp, _i, _f, _vp],
+        "mstar_add_tanh": [_vp, _vp, _vp, _vp, _i, _f, _vp, _i, _i, _i, _vp],
         "mstar_add_rmsnorm": [_vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _f, _i, _vp],
         "mstar_gather_add_rows": [_vp, _vp, _i, _vp, _vp, _i, _i, _vp],
         "mstar_silu_mul": [_vp, _vp, _i, _i, _i, _i, _f, _f, _vp],
@@ -41,14 +43,18 @@ _SIGNATURES = {
     "hyper": {
         "mstar_hyper_step": [_vp, _vp, _vp, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp,
                              _i, _i, _i, _f, _i, _i, _vp],
+        "mstar_hyper_step_tanh": [_vp, _vp, _vp, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _f, _vp,
+                                  _vp, _i, _i, _i, _i, _i, _i, _vp],
         "mstar_weighted_sum2": [_vp, _vp, _vp, _ll, _f, _f, _i, _vp],
     },
     "gated_delta": {
         "mstar_delta_prepare": [_vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp,
                                 _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp],
         "mstar_delta_scan": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _vp, _i, _i, _i, _i,
-                             _i, _i, _vp],
-        "mstar_delta_finish": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _f, _vp],
+                             _i, _i, _i, _vp],
+        "mstar_delta_finish": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _i, _vp],
+        "mstar_delta_scan_head_pieces": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _vp, _vp, _i,
+                                         _i, _i, _i, _i, _i, _i, _vp],
         "mstar_delta_scan_pieces": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _ll, _vp, _vp, _i,
                                     _i, _i, _i, _i, _i, _i, _vp],
     },
@@ -64,7 +70,7 @@ _SIGNATURES = {
                               _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
     },
     "routed_experts": {
-        "mstar_route_topk": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+        "mstar_route_topk": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp],
         "mstar_experts_by_row": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
                                  _i, _i, _f, _f, _vp, _i, _vp],
         "mstar_experts_grouped": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
@@ -73,7 +79,7 @@ _SIGNATURES = {
     "attention_sink": {
         "mstar_sink_prepare": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i,
                                _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp, _i, _i, _vp, _vp,
-                               _vp, _ll, _i, _i, _f, _i, _vp],
+                               _vp, _ll, _i, _i, _f, _i, _vp, _i, _f, _vp],
         "mstar_conv_state_advance": [_vp, _i, _i, _i, _vp, _vp, _vp, _ll, _i, _vp],
         "mstar_sink_attention_generic": [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i,
                                          _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _i, _i, _vp, _vp],

@@ -21,7 +21,8 @@ gate a head on the output; the gate's rows ride in the fused first product.  Fur
 options of that path: an RMS norm over the whole q (and k) projection instead of a head,
 rotary pairs of neighbouring features, a query temperature that grows with the logarithm of
 the position, a tanh soft cap on the scores, a sink in the softmax's denominator (a learned
-number a head, or zero), a sigmoid gate a feature on the heads' outputs, a mask of chunks
+number a head, or zero), a sigmoid gate a feature on the heads' outputs, an RMS norm a head
+without a weight, values blended with those of an earlier layer of the same step, a mask of chunks
 instead of a window (the cache then keeps as many keys as a chunk is long), a learned number
 a head added to the scores, and weights that are sigmoids of the scores instead of a softmax.
 """
@@ -56,7 +57,7 @@ class Attention:
             first = {"qkv.weight": ParamSpec((q_rows + kv_rows, spec.hidden_size))}
             if spec.bias:
                 first["qkv.bias"] = ParamSpec((q_rows + kv_rows,), role="vector", init="zeros")
-        if spec.qk_norm_eps is not None:
+        if spec.qk_norm_eps is not None and spec.qk_norm_weight:
             per_q, per_k = (spec.num_heads, spec.num_kv_heads) if spec.qk_norm_whole else (1, 1)
             first["q_norm.weight"] = ParamSpec((per_q * spec.head_dim,), role="vector", init="ones")
             first["k_norm.weight"] = ParamSpec((per_k * spec.head_dim,), role="vector", init="ones")
@@ -68,6 +69,8 @@ class Attention:
             first["q_conv.weight"] = ParamSpec((q_rows, spec.conv_taps), role="vector")
             first["k_conv.weight"] = ParamSpec((spec.num_kv_heads * spec.head_dim, spec.conv_taps),
                                                role="vector")
+        if spec.value_mix == "blend":
+            first["value_mix"] = ParamSpec((1,), role="vector")
         first["o.weight"] = ParamSpec((spec.hidden_size, spec.num_heads * spec.value_dim))
         return first
 
@@ -107,6 +110,13 @@ class Attention:
         if spec.qk_norm_whole and (spec.conv_taps or spec.qk_norm_eps is None):
             raise ValueError("a norm over the whole projection needs qk_norm_eps and no "
                              "convolution")
+        if spec.value_mix not in (None, "first", "blend"):
+            raise ValueError(f"value_mix {spec.value_mix!r} is not known (first, blend)")
+        if spec.value_mix and spec.value_from_key:
+            raise ValueError("values that are keys are not blended")
+        self.value_lam = None
+        if spec.value_mix == "blend":
+            self.value_lam = float(params["value_mix"].float().reshape(()).item())
         if spec.sink not in (None, "learned", "zero"):
             raise ValueError(f"sink {spec.sink!r} is not known (learned, zero)")
         self.sink = None
@@ -170,13 +180,23 @@ class Attention:
         conv = None
         if s.conv_taps:
             conv = (self.q_conv, self.k_conv, ctx.qo_indptr, ctx.slots, cache.state)
+        first_values = None
+        if s.value_mix is not None:
+            v0 = (s.num_heads + s.num_kv_heads) * s.head_dim
+            if s.value_mix == "first":
+                if self.bias is not None:
+                    raise ValueError("the values handed on are those of a projection without bias")
+                ctx.extras["first_values"] = qkv[:, v0:v0 + s.num_kv_heads * s.value_dim]
+            else:
+                first_values = (ctx.extras["first_values"], self.value_lam)
         q = ops.sink_prepare(qkv, self.bias, self.q_norm, self.k_norm, self.freq, ctx.positions,
                              ctx.cache_pos, ctx.token_req, cache.block_table, cache.kv,
                              s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, self.rot,
                              cache.page_size, s.qk_norm_eps or 0.0, self.runtime.dtype,
                              conv=conv, value_from_key=s.value_from_key,
                              interleaved=s.position.interleaved and self.rot > 0,
-                             norm_whole=s.qk_norm_whole, q_temp=s.q_temp)
+                             norm_whole=s.qk_norm_whole, q_temp=s.q_temp,
+                             norm=s.qk_norm_eps is not None, first_values=first_values)
         if s.conv_taps > 1:
             ops.conv_state_advance(qkv, (s.num_heads + s.num_kv_heads) * s.head_dim, s.conv_taps,
                                    ctx.qo_indptr, ctx.slots, cache.state, ctx.num_entries)

@@ -156,6 +156,16 @@ class ResidualStream:
             return d.gather_rows(self.h, rows)
         return ops.gather_add_rows(self.h, self.take_delta(), rows)
 
+    def gather_normed(self, rows: torch.Tensor, norm) -> torch.Tensor:
+        """The rows asked for, everything pending added, through a norm part: in the launch that
+        gathers them where the residual offers that."""
+        fused = getattr(self.copies, "gather_normed", None)
+        if fused is not None:
+            out = fused(rows, norm)
+            if out is not None:
+                return out
+        return norm.norm_rows(self.gather(rows))
+
     def push(self, delta: torch.Tensor, post=None, scale: float = 1.0) -> None:
         if self.delta is not None:
             raise RuntimeError("a part's output was pushed before the previous one was added")

@@ -164,13 +164,28 @@ class ResidualCopies:
         if not write:                # nothing to write yet: the kernel still wants its tables
             write = dict(zip(("mix", "out"), _no_write_tables(self.x.shape[1], self.x.device)))
         out = ops.hyper_step(self.x, init=self.init, **write, **read)
-        if "rows" not in read:      # a sum leaves the copies as they were
+        if read.get("rows") is None:     # a sum leaves the copies as they were
             self.init = None
             self.pending = None
         return out
 
     def gather(self, rows: torch.Tensor) -> torch.Tensor:
         return self.step(rows=rows)
+
+    def read_through(self, norm, table: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+        """What a sublayer reads: ``norm(sum_s table[s] x_s)`` with the pending write done."""
+        if norm.spec.kind == "dynamic_tanh":
+            # a pending write means that the sublayer's kernels lie between this one and the
+            # one that wrote the copies
+            return self.step(read=table, tanh_norm=norm.kernel_args, out_dtype=dtype,
+                             x_static=self.pending is not None)
+        return self.step(read=table, norm_weight=norm.weight, eps=norm.spec.eps, out_dtype=dtype)
+
+    def gather_normed(self, rows: torch.Tensor, norm):
+        """The rows' sums through the model's last norm in one launch (None: not this norm)."""
+        if norm.spec.kind != "dynamic_tanh":
+            return None
+        return self.step(rows=rows, tanh_norm=norm.kernel_args, out_dtype=norm.runtime.dtype)
 
 
 _NO_WRITE: dict = {}
@@ -240,8 +255,10 @@ class HyperBlock:
             self.tables[q] = (t_in.contiguous(), (t_out * spec.residual_mult).contiguous(),
                               t_mix.contiguous())
         for norm in (self.norm1, self.norm2):
-            if norm is not None and (norm.spec.kind != "rmsnorm" or norm.spec.weight_offset):
-                raise ValueError("a hyper-connection block reads through a plain RMS norm")
+            if norm is not None and (norm.spec.kind not in ("rmsnorm", "dynamic_tanh")
+                                     or norm.spec.weight_offset):
+                raise ValueError("a hyper-connection block reads through a plain RMS norm or a "
+                                 "dynamic tanh")
         self.graph_safe = all(getattr(p, "graph_safe", False) is True for p in self.parts.values())
 
     def _pending(self, y, q: int) -> dict:
@@ -269,12 +286,10 @@ class HyperBlock:
         elif copies.x.shape[1] != self.streams:
             raise ValueError("blocks of one model keep the same number of residual copies")
         dtype = self.runtime.dtype
-        x = copies.step(read=self.tables[1][0], norm_weight=self.norm1.weight,
-                        eps=self.norm1.spec.eps, out_dtype=dtype)
+        x = copies.read_through(self.norm1, self.tables[1][0], dtype)
         copies.pending = self._pending(self.mixer.forward(x, ctx, cache), 1)
         if self.ffn is not None:
-            y = copies.step(read=self.tables[2][0], norm_weight=self.norm2.weight,
-                            eps=self.norm2.spec.eps, out_dtype=dtype)
+            y = copies.read_through(self.norm2, self.tables[2][0], dtype)
             copies.pending = self._pending(self.ffn.forward(y, ctx), 2)
 
 

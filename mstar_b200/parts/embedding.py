@@ -1,8 +1,8 @@
 """Token embedding and LM head parts: the two ends of the residual stream.
 
 "table": h0 = E[ids] (mstar/model/orpheus/components/language_model.py:61-66, no scaling
-there; ``multiplier`` serves architectures that scale the rows), written as the float
-residual.  "linear": logits = x W^T without bias (language_model.py:95-101), float, with an
+there; ``multiplier`` serves architectures that scale the rows, ``norm`` those that norm
+them), written as the float residual.  "linear": logits = x W^T without bias (language_model.py:95-101), float, with an
 optional scale and soft cap.  A tied head is the same tensor under two parameter names;
 the checkpoint map says so, the parts do not know.
 """
@@ -13,7 +13,7 @@ import torch
 from .. import ops
 from ..weights.names import ParamSpec
 from .base import Runtime, StepContext
-from .registry import register_part
+from .registry import build_part, part_class, register_part
 
 
 class TokenEmbedding:
@@ -21,17 +21,30 @@ class TokenEmbedding:
 
     @classmethod
     def param_specs(cls, spec) -> dict:
-        return {"weight": ParamSpec((spec.vocab_size, spec.hidden_size), role="table")}
+        out = {"weight": ParamSpec((spec.vocab_size, spec.hidden_size), role="table")}
+        if spec.norm is not None:
+            for local, ps in part_class("norm", spec.norm).param_specs(spec.norm).items():
+                out[f"norm.{local}"] = ps
+        return out
 
     def __init__(self, spec, params: dict, runtime: Runtime):
         self.spec = spec
         self.weight = params["weight"]
+        self.norm = None
+        if spec.norm is not None:
+            self.norm = build_part("norm", spec.norm, {k[5:]: v for k, v in params.items()
+                                                       if k.startswith("norm.")}, runtime)
+            self.graph_safe = getattr(self.norm, "graph_safe", False) is True
 
     def forward(self, token_ids: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         """Float residual [tokens, hidden]; tokens that only the device holds come through
         ``ctx.token_source``."""
-        return ops.embed_rows(self.weight, token_ids, source=ctx.token_source,
-                              scale=self.spec.multiplier)
+        if self.norm is not None and self.norm.spec.kind == "dynamic_tanh":
+            return ops.embed_tanh(self.weight, token_ids, self.norm.kernel_args,
+                                  source=ctx.token_source, scale=self.spec.multiplier)
+        h = ops.embed_rows(self.weight, token_ids, source=ctx.token_source,
+                           scale=self.spec.multiplier)
+        return h if self.norm is None else self.norm.norm_rows(h, torch.float32)
 
 
 class LinearHead:

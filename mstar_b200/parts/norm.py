@@ -1,4 +1,4 @@
-"""RMSNorm part, fused with the residual add that precedes it.
+"""Norm parts, fused with the residual add that precedes them: RMS norm and dynamic tanh.
 
 out = x * rsqrt(mean(x^2) + eps) * (weight + weight_offset), x the float residual
 after adding the pending part output.  Llama mode multiplies by ``weight``
@@ -6,6 +6,8 @@ after adding the pending part output.  Llama mode multiplies by ``weight``
 form the reference calls gemma_mode (norm.py:46-52).  The reference down-casts
 float input to bfloat16 before the library norm (mstar/utils/flashinfer_utils.py:
 38-40); here sums and the scale are float in both dtypes.
+
+Dynamic tanh: out = tanh(alpha * x) * weight + bias, elementwise, float inside.
 """
 from __future__ import annotations
 
@@ -69,11 +71,58 @@ class RMSNorm:
         return ops.add_rmsnorm(stream.h, delta, self.weight, self.spec.eps, self.runtime.dtype,
                                self.spec.weight_offset, resid_static=delta is not None)
 
-    def norm_rows(self, rows_f32: torch.Tensor) -> torch.Tensor:
+    def norm_rows(self, rows_f32: torch.Tensor, dtype=None) -> torch.Tensor:
         """Norm of float rows that carry no pending delta (the final norm on the
         gathered rows)."""
-        return ops.add_rmsnorm(rows_f32, None, self.weight, self.spec.eps, self.runtime.dtype,
-                               self.spec.weight_offset)
+        return ops.add_rmsnorm(rows_f32, None, self.weight, self.spec.eps,
+                               dtype or self.runtime.dtype, self.spec.weight_offset)
 
 
+class DynamicTanh:
+    """tanh(alpha * x) * weight + bias with one learned alpha; no mean, no variance."""
+
+    graph_safe = True
+
+    @classmethod
+    def param_specs(cls, spec) -> dict:
+        return {"weight": ParamSpec(shape=(spec.size,), role="vector", init="ones"),
+                "bias": ParamSpec(shape=(spec.size,), role="vector", init="zeros"),
+                "alpha": ParamSpec(shape=(1,), role="vector", init="ones")}
+
+    def __init__(self, spec, params: dict, runtime: Runtime):
+        self.spec = spec
+        self.runtime = runtime
+        self.weight, self.bias = params["weight"], params["bias"]
+        if self.weight.dtype != self.bias.dtype:        # the kernels take them in one type
+            self.weight, self.bias = self.weight.float(), self.bias.float()
+        self.weight, self.bias = self.weight.contiguous(), self.bias.contiguous()
+        for name in ("weight", "bias"):
+            if tuple(getattr(self, name).shape) != (spec.size,):
+                raise ValueError(f"dynamic_tanh {name} has shape "
+                                 f"{tuple(getattr(self, name).shape)}, expected ({spec.size},)")
+        self.alpha = float(params["alpha"].float().reshape(()).item())
+
+    @property
+    def kernel_args(self) -> tuple:
+        """What the kernels that apply this norm on the way take: (weight, bias, alpha)."""
+        return self.weight, self.bias, self.alpha
+
+    def add_normed(self, resid, delta, scale: float = 1.0, rows_dtype=None):
+        """resid += scale * norm(delta), with ``rows_dtype`` also as rows of that dtype."""
+        d = ops.add_tanh(ops.convert(delta, torch.float32), None, self.kernel_args, torch.float32)
+        resid.add_(d, alpha=scale)
+        return None if rows_dtype is None else ops.convert(resid, rows_dtype)
+
+    def add_norm(self, stream: ResidualStream) -> torch.Tensor:
+        """Fold the pending delta into the residual and return the normed rows."""
+        delta = stream.take_delta()
+        if delta is not None:
+            delta = ops.convert(delta, self.runtime.dtype)
+        return ops.add_tanh(stream.h, delta, self.kernel_args, self.runtime.dtype)
+
+    def norm_rows(self, rows_f32: torch.Tensor, dtype=None) -> torch.Tensor:
+        return ops.add_tanh(rows_f32, None, self.kernel_args, dtype or self.runtime.dtype)
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "rmsnorm", RMSNorm)

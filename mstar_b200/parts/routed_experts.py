@@ -2,7 +2,8 @@
 feed-forwards per token; an optional shared one runs for every token and is added.
 
 The router's logits are a product with float output; a kernel turns them into the chosen
-experts and their weights (sigmoid or softmax scores, renormalised or not).  The shared
+experts and their weights (sigmoid or softmax scores, a correction for the choice, groups of
+which the best stay eligible, renormalised and scaled or not).  The shared
 expert is the dense gated feed-forward's path (one fused gate/up product, one down
 product); the routed experts' kernels add its output while they write theirs, times the
 sigmoid of a gate a token where it has one (a further row of the router's product).  A few rows
@@ -76,7 +77,9 @@ class RoutedExperts:
         shared_gate = logits[:, self.outputs:self.outputs + 1] if s.shared_gate else None
         logits = logits[:, :self.outputs]
         chosen, weight = ops.route_topk(logits, s.top, softmax=s.score == "softmax",
-                                        renormalize=s.renormalize, choice_bias=self.correction)
+                                        renormalize=s.renormalize, choice_bias=self.correction,
+                                        groups=s.groups, renorm_eps=s.renorm_eps,
+                                        weight_scale=s.weight_scale)
         shared = None
         if self.shared_gate_up is not None:
             shared = ops.linear(ops.gated_up(x, self.shared_gate_up, static_weights=True,

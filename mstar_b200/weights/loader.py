@@ -178,7 +178,7 @@ def load_parameters(source, param_specs: Mapping[str, ParamSpec],
                     missing.append(s.name)
                 continue
             got, _ = ckpt.shape_dtype(s.name)
-            want = (s.rows,) + tuple(spec.shape[1:])
+            want = s.checkpoint_shape(spec.shape)
             if got != want:
                 wrong_shape.append((s.name, got, want))
         covered = sum(s.rows for s in sources)

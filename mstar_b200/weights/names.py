@@ -32,12 +32,17 @@ class ParamSpec:
 
 @dataclass(frozen=True)
 class TensorSource:
-    """Checkpoint tensor ``name`` fills ``rows`` rows of ``param`` from ``row_start``."""
+    """Checkpoint tensor ``name`` fills ``rows`` rows of ``param`` from ``row_start``.
+    ``scalar``: the checkpoint's tensor has no dimension and is one number of ``param``."""
 
     name: str
     param: str
     row_start: int
     rows: int
+    scalar: bool = False
+
+    def checkpoint_shape(self, param_shape: tuple) -> tuple:
+        return () if self.scalar else (self.rows,) + tuple(param_shape[1:])
 
 
 @dataclass

@@ -29,7 +29,7 @@ def checkpoint_tensor_shapes(config: ModelConfig, param_specs: Mapping[str, Para
         if src.name in cmap.optional:
             continue
         spec = param_specs[src.param]
-        out[src.name] = ((src.rows,) + tuple(spec.shape[1:]), spec)
+        out[src.name] = (src.checkpoint_shape(spec.shape), spec)
     return out
 
 
