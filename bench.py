@@ -5,7 +5,7 @@ one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--rounds R] [--page-size P]
                     [--impl ours|reference] [--workloads all|none|mixed64|long8]
-    python bench.py --arch tifosun|vudivik|relurax|mokotar|sokalorn [--arch-size small|medium]   (another architecture)
+    python bench.py --arch tifosun|vudivik|relurax|mokotar|sokalorn|famarax [--arch-size small|medium]   (another architecture)
 
 One JSON line on stdout.  ``value``: decoded tokens per second of the engine's step
 function plus greedy sampling, timed on the device with CUDA events: W warm-up steps, then
@@ -428,6 +428,8 @@ def arch_bench(args) -> int:
         return mokotar_bench(args)
     if args.arch == "sokalorn":
         return sokalorn_bench(args)
+    if args.arch == "famarax":
+        return famarax_bench(args)
     pk = peaks()
     t_cfg, l_cfg = tifosun_sizes(args.arch_size)
     page, batch = args.page_size, args.batch
@@ -1511,6 +1513,244 @@ def sokalorn_bench(args) -> int:
     return 0
 
 
+# ------------------------------------------------------------------ a sixth architecture
+def famarax_sizes(name: str) -> tuple:
+    """(Famarax config, Mokotar config, Llama config) at layer sizes that resemble a real model's:
+    three delta-rule layers to one attention in a window, four copies of the residual, experts
+    in groups beside a shared one in every layer.  The Mokotar beside it, the closest decoder of
+    this engine (hyper-connections, a soft-capped attention, a gated delta rule), and the Llama
+    have the same width, depth, vocabulary, heads and key/value heads."""
+    if name == "small":
+        width, depth, vocab = 1024, 8, 32000
+        heads, kv_heads, experts, top, groups, ff, shared = 8, 2, 16, 2, (4, 2), 512, 1024
+    elif name == "medium":
+        width, depth, vocab = 2048, 12, 64000
+        heads, kv_heads, experts, top, groups, ff, shared = 16, 4, 32, 4, (8, 4), 512, 2048
+    else:
+        raise ValueError(f"unknown size {name!r} (small, medium)")
+    att = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0,
+               mask={"size": 1024}, rot={"base": 500000.0, "dims": 128}, v_mix=True)
+    delta = dict(heads=heads, kv_heads=heads // 2, dim=128, vdim=128, conv=4)
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0,
+                                     "groups": {"count": groups[0], "keep": groups[1]}},
+           "expert": {"ff": ff}, "shared": {"ff": shared}}
+    layers = [{"type": "attention" if i % 4 == 3 else "delta",
+               "mixer": json.loads(json.dumps(att if i % 4 == 3 else delta)), "mlp": moe}
+              for i in range(depth)]
+    famarax = {"architecture": "Famarax", "width": width, "vocab": vocab, "norm": {"eps": 1e-6},
+               "streams": 4, "logit_scale": 0.5, "logit_softcap": 30.0, "layers": layers}
+    mokotar, _, _ = mokotar_sizes(name)
+    llama = dict(ORPHEUS_3B, num_hidden_layers=depth, hidden_size=width,
+                 num_attention_heads=heads, num_key_value_heads=kv_heads, head_dim=128,
+                 intermediate_size=top * ff + shared, vocab_size=vocab, tie_word_embeddings=False)
+    return famarax, mokotar, llama
+
+
+def famarax_bench(args) -> int:
+    """``--arch famarax``: prefill and decode throughput of the Famarax decoder (random weights,
+    bfloat16) beside the Mokotar and Llama decoders at equal size, through the same step function;
+    then its kernels alone at the sizes of one layer, each beside the like kernel of the closest
+    decoder (the delta rule with one decay a head, its input and its gate: Mokotar's with a decay a
+    channel; the hyper-connection kernel through a dynamic tanh: Mokotar's through an RMS norm; the
+    capped window attention and its input kernel: Mokotar's attention over every key, Vudivik's
+    window; the grouped choice and the experts: Sokalorn's), with what each has to move against the
+    measured peaks.  ``--arch-parts kernels|models``: one half only.  One JSON line."""
+    import torch
+
+    from mstar_b200 import ops
+    from mstar_b200.parts.base import StepContext
+
+    pk = peaks()
+    f_cfg, m_cfg, l_cfg = famarax_sizes(args.arch_size)
+    page, batch = args.page_size, args.batch
+    out = {"arch": "Famarax", "size": args.arch_size, "batch": batch, "prompt_len": PROMPT_LEN,
+           "peaks": pk["source"], "models": {}, "kernels": {}}
+    if args.arch_parts != "kernels":
+        _time_models(args, (("famarax", f_cfg), ("mokotar", m_cfg), ("llama", l_cfg)), out)
+    if args.arch_parts == "models":
+        print(json.dumps(out))
+        return 0
+
+    dev = "cuda:0"
+    g = torch.Generator(device=dev).manual_seed(0)
+
+    def rnd(*shape, scale=1.0):
+        return (scale * torch.randn(*shape, generator=g, device=dev)).to(torch.bfloat16)
+
+    def f32(*shape):
+        return torch.randn(*shape, generator=g, device=dev)
+
+    def i32(v):
+        return torch.tensor(v, dtype=torch.int32, device=dev)
+
+    def record(name, ms, nbytes=None, flops=None, **more):
+        row = {"ms": round(ms, 4)}
+        if nbytes is not None:
+            row["gbs"] = round(nbytes / ms / 1e6, 1)
+            row["frac_hbm"] = round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4)
+        if flops is not None:
+            row["tflops"] = round(flops / ms / 1e9, 2)
+            row["frac_bf16"] = round(flops / ms / 1e9 / pk["bf16_tflops"], 5)
+        row.update(more)
+        out["kernels"][name] = row
+
+    width, vocab = f_cfg["width"], f_cfg["vocab"]
+    att, delta, moe = f_cfg["layers"][3]["mixer"], f_cfg["layers"][0]["mixer"], f_cfg["layers"][0]["mlp"]
+    H, G, hd, window = att["heads"], att["kv_heads"], att["dim"], att["mask"]["size"]
+    ctx_len = PROMPT_LEN
+    pages_per = -(-ctx_len // page)
+    for tokens, reqs, label in ((batch, batch, "decode"), (PROMPT_LEN, 1, "prefill")):
+        per = tokens // reqs
+        copies = 1 if label == "prefill" else max(1, -(-(160 << 20) // (reqs * ctx_len * G * hd * 4)))
+        caches = [rnd(reqs * pages_per + 1, 2, G, page, hd).view(reqs * pages_per + 1, -1)
+                  for _ in range(copies)]
+        table = torch.randperm(reqs * pages_per, device=dev).to(torch.int32).view(reqs, pages_per)
+        token_req = i32([r for r in range(reqs) for _ in range(per)])
+        cache_pos = i32([ctx_len - per + k for _ in range(reqs) for k in range(per)])
+        indptr = i32([k * per for k in range(reqs + 1)])
+        slots = i32(list(range(reqs)))
+        sc = StepContext(num_tokens=tokens, num_entries=reqs, token_req=token_req,
+                         positions=cache_pos, cache_pos=cache_pos, qo_indptr=indptr,
+                         kv_len=i32([ctx_len] * reqs), slots=slots, q_lens=[per] * reqs,
+                         kv_lens=[ctx_len] * reqs, host_slots=list(range(reqs)), max_q_len=per,
+                         max_kv_len=ctx_len, num_decode=reqs if per == 1 else 0)
+        reps = max(copies, 4) if label == "decode" else 2
+        turn = {"i": 0}
+
+        def rotated(items):
+            turn["i"] += 1
+            return items[turn["i"] % len(items)]
+
+        # attention and its input kernel
+        q, rows = rnd(tokens, H * hd), (H + 2 * G) * hd
+        qkv = f32(tokens, rows + H * hd)                        # (the gate's columns: Mokotar's form)
+        sink = f32(H)
+        keys = sum(ctx_len - per + k + 1 for k in range(per)) * reqs
+        wkeys = sum(min(ctx_len - per + k + 1, window) for k in range(per)) * reqs
+        kv_bytes = G * hd * 4.0 * reqs
+        seen = min(ctx_len, window if per == 1 else ctx_len)
+        ms = _time_graph(lambda: ops.sink_attention(
+            q, rotated(caches), table, token_req, cache_pos, H, G, hd, hd, page, window, 0, att["scale"],
+            ctx=sc, softcap=att["softcap"]), reps=reps)
+        record(f"capped_window_attention_{label}", ms, nbytes=kv_bytes * seen, flops=4.0 * H * wkeys * hd)
+        ms = _time_graph(lambda: ops.sink_attention(
+            q, rotated(caches), table, token_req, cache_pos, H, G, hd, hd, page, window, 4,
+            att["scale"], ctx=sc), reps=reps)
+        record(f"vudivik_window_attention_{label}", ms, nbytes=kv_bytes * (seen + 4 if per == 1 else seen),
+               flops=4.0 * H * (wkeys + 4 * tokens) * hd)
+        ms = _time_graph(lambda: ops.sink_attention(
+            q, rotated(caches), table, token_req, cache_pos, H, G, hd, hd, page, 0, 0, att["scale"],
+            ctx=sc, gate=qkv[:, rows:], softcap=att["softcap"], sink=sink), reps=reps)
+        record(f"mokotar_attention_{label}", ms, nbytes=kv_bytes * ctx_len, flops=4.0 * H * keys * hd)
+        freq = torch.rand(hd // 2, dtype=torch.float64, device=dev)
+        first = f32(tokens, G * hd)
+        io_bytes = tokens * (rows * 4 + H * hd * 2 + 2 * G * hd * 2.0)
+        ms = _time_graph(lambda: ops.sink_prepare(
+            qkv, None, None, None, freq, cache_pos, cache_pos, token_req, table, caches[0], H, G, hd,
+            hd, hd, page, 1e-6, torch.bfloat16, norm=True, first_values=(first, 0.4)), reps=8)
+        record(f"rope_norm_blend_cache_{label}", ms, nbytes=io_bytes + tokens * G * hd * 4.0)
+        nq, nk = rnd(hd), rnd(hd)
+        ms = _time_graph(lambda: ops.sink_prepare(
+            qkv, None, nq, nk, None, cache_pos, cache_pos, token_req, table, caches[0], H, G, hd, hd, 0,
+            page, 1e-6, torch.bfloat16, q_temp=(0.3, 512)), reps=8)
+        record(f"mokotar_norm_temperature_cache_{label}", ms, nbytes=io_bytes)
+
+        # the delta rule with one decay a head, beside a decay a channel, at the same sizes
+        DH, DG, D, VD, taps = (delta[k] for k in ("heads", "kv_heads", "dim", "vdim", "conv"))
+        channels = 2 * DG * D + DH * VD
+        size = ops.gated_delta_state_size(DH, DG, D, VD, taps)
+        n_state = max(1, -(-(160 << 20) // (reqs * size * 4))) if label == "decode" else 1
+        states = [torch.zeros(reqs, size, device=dev) for _ in range(n_state)]
+        proj, conv_w = f32(tokens, channels + 2 * DH + DH * VD), rnd(channels, taps)
+        a_exp = torch.rand(DH, device=dev) + 0.5
+        sreps = max(n_state, 4) if label == "decode" else 2
+        for name, a_proj, decays in (("head_decay", None, DH), ("mokotar", f32(tokens, DH * D), DH * D)):
+            dt_bias = f32(decays) - 4.0
+            prep = lambda: ops.delta_prepare(proj, conv_w, a_proj, dt_bias, a_exp, token_req, indptr,
+                                             slots, states[0], DH, DG, D, VD, taps, 1e-6)
+            ms = _time_graph(prep, reps=8)
+            record(f"{name}_delta_conv_unit_decay_{label}", ms,
+                   nbytes=tokens * 2.0 * (channels + DH + decays) * 4)
+            pre = prep()
+            ms = _time_graph(lambda: ops.delta_scan(*pre, indptr, slots, rotated(states), reqs, DH, DG, D,
+                                                    VD, taps, max_q_len=per), reps=sreps)
+            record(f"{name}_delta_scan_{label}", ms,
+                   nbytes=reqs * DH * D * VD * 8.0 + tokens * (2 * DG * D + 2 * DH * VD + DH + decays) * 4.0,
+                   tokens_per_us=round(per / ms / 1e3, 3),
+                   fp32_tflops=round(8.0 * tokens * DH * D * VD / ms / 1e9, 2))
+        ms = _time_graph(lambda: ops.conv_state_advance(proj, channels, taps, indptr, slots, states[0],
+                                                        reqs), reps=8)
+        record(f"conv_state_advance_{label}", ms, nbytes=reqs * (taps - 1) * channels * 8.0)
+        o, nw, gate = f32(tokens, DH * VD), f32(VD), rnd(tokens, DH * VD)
+        ms = _time_graph(lambda: ops.delta_finish(o, proj[:, channels + 2 * DH:], nw, DH, VD, 1e-6,
+                                                  torch.bfloat16, 1.0, "silu"), reps=8)
+        record(f"delta_norm_silu_gate_{label}", ms, nbytes=tokens * DH * VD * 10.0)
+        ms = _time_graph(lambda: ops.delta_finish(o, gate, nw, DH, VD, 1e-6, torch.bfloat16), reps=8)
+        record(f"mokotar_delta_norm_gate_{label}", ms, nbytes=tokens * DH * VD * 8.0)
+
+        # between the sublayers, and the model's ends
+        S = f_cfg["streams"]
+        w, b = rnd(width), rnd(width)
+        tanh_norm = (w, b, 0.7)
+        # rotated over more than L2 where a prompt's copies alone do not exceed it
+        xs = [f32(tokens, S, width) for _ in range(max(1, -(-(300 << 20) // (tokens * S * width * 4)))
+                                                   if label == "prefill" else 1)]
+        y = rnd(tokens, width)
+        mix = torch.eye(S, device=dev).contiguous()
+        t_out, t_in = torch.ones(S, device=dev), torch.full((S,), 1.0 / S, device=dev)
+        hyper_bytes = tokens * width * (8.0 * S + 2 + 2)
+        ms = _time_graph(lambda: ops.hyper_step(rotated(xs), y=y, mix=mix, out=t_out, read=t_in,
+                                                tanh_norm=tanh_norm, out_dtype=torch.bfloat16,
+                                                x_static=label == "prefill"), reps=20)
+        record(f"hyper_write_read_tanh_{label}", ms, nbytes=hyper_bytes)
+        ms = _time_graph(lambda: ops.hyper_step(rotated(xs), y=y, mix=mix, out=t_out, read=t_in,
+                                                norm_weight=w, eps=1e-6, out_dtype=torch.bfloat16), reps=20)
+        record(f"mokotar_hyper_write_read_norm_{label}", ms, nbytes=hyper_bytes)
+        embed, ids = rnd(vocab, width), torch.randint(0, vocab, (tokens,), device=dev, dtype=torch.int32)
+        ms = _time_graph(lambda: ops.embed_tanh(embed, ids, tanh_norm), reps=20)
+        record(f"embed_tanh_{label}", ms, nbytes=tokens * width * 6.0)
+        ms = _time_graph(lambda: ops.embed_rows(embed, ids), reps=20)
+        record(f"embed_rows_{label}", ms, nbytes=tokens * width * 6.0)
+        last = i32([(r + 1) * per - 1 for r in range(reqs)])
+        ms = _time_graph(lambda: ops.hyper_step(xs[0], y=y, mix=mix, out=t_out, rows=last,
+                                                tanh_norm=tanh_norm, out_dtype=torch.bfloat16), reps=20)
+        record(f"sum_of_copies_tanh_{label}", ms, nbytes=reqs * width * (4.0 * S + 4))
+        logits = f32(reqs, vocab)
+        ms = _time_graph(lambda: ops.scale_softcap(logits, 0.5, 30.0), reps=20)
+        record(f"logit_scale_softcap_{label}", ms, nbytes=reqs * vocab * 8.0)
+
+        # experts: the grouped choice beside the plain one, silu experts beside the clamped ones
+        E, top, ff, sff = (moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"],
+                           moe["shared"]["ff"])
+        groups = (moe["router"]["groups"]["count"], moe["router"]["groups"]["keep"])
+        z, corr = f32(tokens, E), f32(E) * 0.02
+        grouped = lambda: ops.route_topk(z, top, softmax=True, renormalize=True, choice_bias=corr,
+                                         groups=groups, renorm_eps=1e-20, weight_scale=2.0)
+        ms = _time_graph(grouped, reps=20)
+        record(f"grouped_choice_{label}", ms, nbytes=tokens * (E * 4.0 + top * 8))
+        ms = _time_graph(lambda: ops.route_topk(z, top, softmax=True, renormalize=True,
+                                                choice_bias=corr), reps=20)
+        record(f"plain_choice_{label}", ms, nbytes=tokens * (E * 4.0 + top * 8))
+        chosen, weight = grouped()
+        ncopies = max(1, -(-(160 << 20) // (E * 3 * ff * width * 2)))
+        w_gu = [rnd(E * 2 * ff, width, scale=0.02) for _ in range(ncopies)]
+        w_dn = [rnd(E * width, ff, scale=0.02) for _ in range(ncopies)]
+        x, add = rnd(tokens, width), rnd(tokens, width)
+        used = len(set(chosen.flatten().tolist()))
+        for name, clamp in (("experts", None), ("sokalorn_clamped_experts", (7.0, 1.702))):
+            def experts():
+                i = turn["i"] = turn["i"] + 1
+                return ops.routed_experts(x, w_gu[i % ncopies], w_dn[i % ncopies], chosen, weight, E, ff,
+                                          False, add=add, clamp=clamp)
+
+            ms = _time_graph(experts, reps=max(ncopies * 2, 4) if label == "decode" else 2)
+            record(f"{name}_{label}", ms, nbytes=used * 3.0 * ff * width * 2,
+                   flops=2.0 * tokens * top * 3 * ff * width, experts_used=used)
+    ops.check_error_word(dev)
+    print(json.dumps(out))
+    return 0
+
+
 # --------------------------------------------------------------- single kernels
 def _time_graph(fn, reps: int = 20, rounds: int = 5) -> float:
     """Median milliseconds of one call of ``fn`` when ``reps`` calls are replayed as one
@@ -1754,10 +1994,12 @@ def main() -> int:
     ap.add_argument("--small", action="store_true", help="a smaller case, for profiler captures")
     ap.add_argument("--sizes", default="orpheus-3b", choices=sorted(SIZES),
                     help="layer sizes; the default is the benchmark model")
-    ap.add_argument("--arch", default=None, choices=["tifosun", "vudivik", "relurax", "mokotar", "sokalorn"],
+    ap.add_argument("--arch", default=None, choices=["tifosun", "vudivik", "relurax", "mokotar", "sokalorn", "famarax"],
                     help="measure another architecture beside the Llama decoder at equal size "
                          "(prefill, decode, its own kernels) instead of the headline workload")
     ap.add_argument("--arch-size", default="small", choices=["small", "medium"])
+    ap.add_argument("--arch-parts", default="all", choices=["all", "models", "kernels"],
+                    help="with --arch famarax: the models' throughput, the kernels alone, or both")
     args = ap.parse_args()
     model_name, sizes = SIZES[args.sizes]
     PAGE_SIZE = page = args.page_size
