@@ -1673,14 +1673,11 @@ def famarax_bench(args) -> int:
                    nbytes=tokens * 2.0 * (channels + DH + decays) * 4)
             pre = prep()
             ms = _time_graph(lambda: ops.delta_scan(*pre, indptr, slots, rotated(states), reqs, DH, DG, D,
-                                                    VD, taps, max_q_len=per), reps=sreps)
+                                                    VD, taps, max_q_len=per, conv_rows=proj), reps=sreps)
             record(f"{name}_delta_scan_{label}", ms,
                    nbytes=reqs * DH * D * VD * 8.0 + tokens * (2 * DG * D + 2 * DH * VD + DH + decays) * 4.0,
                    tokens_per_us=round(per / ms / 1e3, 3),
                    fp32_tflops=round(8.0 * tokens * DH * D * VD / ms / 1e9, 2))
-        ms = _time_graph(lambda: ops.conv_state_advance(proj, channels, taps, indptr, slots, states[0],
-                                                        reqs), reps=8)
-        record(f"conv_state_advance_{label}", ms, nbytes=reqs * (taps - 1) * channels * 8.0)
         o, nw, gate = f32(tokens, DH * VD), f32(VD), rnd(tokens, DH * VD)
         ms = _time_graph(lambda: ops.delta_finish(o, proj[:, channels + 2 * DH:], nw, DH, VD, 1e-6,
                                                   torch.bfloat16, 1.0, "silu"), reps=8)

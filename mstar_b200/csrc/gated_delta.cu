@@ -16,10 +16,13 @@
 //   finish   o / rms(o per head) * weight * sigmoid(gate) (or silu(gate)), handed on in the
 //            activation type.
 //
+// The scans also move the slot's convolution inputs on (they run after prepare has read them).
+//
 // A slot is [(taps - 1) * (2 G D + H VD) convolution inputs | S^T as [H][VD][D]], float.
 // Everything here is float whatever the activation type.
 #include "common.cuh"
 #include "mma_util.cuh"
+#include "tma_util.cuh"
 
 // ------------------------------------------------------------------ prepare
 struct DeltaPrepArgs {
@@ -245,6 +248,28 @@ MSTAR_API int mstar_delta_prepare(const float* proj, int row_stride, const void*
 #define GD_ROWS 16          // most rows of a column that one lane keeps
 #define GD_CHUNK 16         // tokens staged at a time
 
+// The convolutions' rows in a slot move on with the scan: the last taps - 1 rows of the sequence's
+// projected channels (a portion shorter than that keeps the newer part of what the slot held).
+struct ConvAdvance {
+    const float* raw;           // null: not here; else the projected rows of the batch's tokens
+    int raw_ld, channels, taps;
+};
+
+// Oldest row first: row s is read from s + n, which is written later or not at all.  Only a head's first
+// block does this (for its share of the channels), so that the others end without that latency.
+__device__ __forceinline__ void gd_advance_conv(const ConvAdvance& c, unsigned long long waited, float* slot,
+                                                int start, int n, int h, int H) {
+    if (c.raw == nullptr || blockIdx.z != 0) return;
+    const float* raw = pdl_after(c.raw, waited);
+    const int keep = c.taps - 1, share = (c.channels + H - 1) / H, end = min(c.channels, (h + 1) * share);
+    for (int ch = h * share + threadIdx.x; ch < end; ch += blockDim.x)
+        for (int s = 0; s < keep; ++s) {
+            const int src = n - keep + s;
+            slot[(size_t)s * c.channels + ch] = src >= 0 ? raw[(size_t)(start + src) * c.raw_ld + ch]
+                                                         : slot[(size_t)(s + n) * c.channels + ch];
+        }
+}
+
 struct DeltaScanArgs {
     const float* q;
     const float* k;
@@ -258,6 +283,7 @@ struct DeltaScanArgs {
     long long state_offset;
     float* out;                 // [tokens][H*VD]
     int H, G, D, VD, chunk;
+    ConvAdvance conv;
 };
 
 __device__ __forceinline__ void gd_copy4(float* dst, const float* src) {
@@ -426,13 +452,15 @@ __global__ void __launch_bounds__(GD_THREADS) delta_scan_kernel(DeltaScanArgs a)
             if (r < D) s_col[r] = s[i];
         }
     }
+    gd_advance_conv(a.conv, waited, state + (size_t)a.slots[e] * a.state_stride, start, n, h, a.H);
 }
 
 MSTAR_API int mstar_delta_scan(const float* q, const float* k, const float* v, const float* beta,
                                const float* decay, const int* qo_indptr, const int* slots,
                                float* state, long long state_stride, long long state_offset,
                                float* out, int entries, int max_q_len, int H, int G, int D, int VD,
-                               int head_decay, void* stream) {
+                               int head_decay, const float* conv_raw, int conv_ld, int channels,
+                               int taps, void* stream) {
     if (entries <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || VD <= 0 || D > 32 * GD_ROWS) return -1;
     if (H > 65535) return -1;
@@ -456,7 +484,7 @@ MSTAR_API int mstar_delta_scan(const float* q, const float* k, const float* v, c
         chunk /= 2;
     const size_t smem = 2 * chunk * per_tok * sizeof(float);
     DeltaScanArgs a{q, k, v, beta, decay, qo_indptr, slots, state, state_stride, state_offset, out,
-                    H, G, D, VD, chunk};
+                    H, G, D, VD, chunk, {taps > 1 ? conv_raw : nullptr, conv_ld, channels, taps}};
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(entries, H, (VD + cols - 1) / cols);
     if (grid.z > 65535) return -1;
@@ -615,6 +643,7 @@ struct DeltaChunkArgs {
     long long state_offset;
     float* out;
     int H, VD, max_pieces, tokens;
+    ConvAdvance conv;
 };
 
 #define GC_THREADS 256
@@ -794,6 +823,7 @@ __global__ void __launch_bounds__(GC_THREADS) delta_scan_pieces_kernel(DeltaChun
     }
     cp_async_wait<0>();
     if (live) gc_store<R>(s_col + lane * R, s);
+    gd_advance_conv(a.conv, waited, state + (size_t)a.slots[e] * a.state_stride, start, n, h, a.H);
 }
 
 // The scan in pieces, for key sizes of 32, 64, 128 or 256 (whole accesses a lane): `work` holds
@@ -804,6 +834,7 @@ MSTAR_API int mstar_delta_scan_pieces(const float* q, const float* k, const floa
                                       const int* slots, float* state, long long state_stride,
                                       long long state_offset, float* out, float* work, int tokens,
                                       int entries, int max_q_len, int H, int G, int D, int VD,
+                                      const float* conv_raw, int conv_ld, int channels, int taps,
                                       void* stream) {
     if (entries <= 0 || tokens <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || VD <= 0) return -1;
@@ -821,7 +852,8 @@ MSTAR_API int mstar_delta_scan_pieces(const float* q, const float* k, const floa
     int code = launch_status();
     if (code != 0) return code;
     DeltaChunkArgs c{p.kt, p.qt, p.kh, p.pc, p.A, p.B, v, beta, qo_indptr, slots, state,
-                     state_stride, state_offset, out, H, VD, max_pieces, tokens};
+                     state_stride, state_offset, out, H, VD, max_pieces, tokens,
+                     {taps > 1 ? conv_raw : nullptr, conv_ld, channels, taps}};
     const int per_buf = 3 * GC_TOKENS * D + 2 * GC_TOKENS * (GC_TOKENS + 1) + GC_TOKENS * GC_COLS +
                         GC_TOKENS + D;
     const size_t smem2 = ((size_t)2 * per_buf + (size_t)GC_COLS * D) * sizeof(float);
@@ -854,11 +886,14 @@ MSTAR_API int mstar_delta_scan_pieces(const float* q, const float* k, const floa
 //   T = (I + L)^-1 diag(beta),   u = T c,   o_t = P_t q_t . S0 + (B T c)_t,
 //   S_C = P_C S0 + sum_j dec(C, j) k_j u_j.
 // A first kernel makes T, B T, P and dec(C, .) for all pieces and heads side by side (products of
-// decays only, never a quotient); the products of keys and queries among themselves are shared by
-// the heads of a group.  The scan reads the q and k rows as they are, several columns a warp, and
-// has no chain from token to token inside a piece.  All float.
-#define GH_WARPS 4
+// decays only, never a quotient; the products of keys and queries among themselves are shared by
+// the heads of a group) and lays them, and the piece's k and q rows, down as the scan wants them in
+// its shared memory, so that a piece is two bulk copies.  The scan has no chain from token to token
+// inside a piece.  All float.
+#define GH_THREADS 128
+#define GH_WAIT_CODE 18             // what the error word gets when a wait for a piece ran out
 #define GH_LD (GC_TOKENS + 4)       // floats between the rows of a C x C matrix in shared memory
+#define GH_MROW (2 * GC_TOKENS + 4) // a token's row of T, of B T, then P_t and dec(C, t)
 
 struct DeltaHeadArgs {
     const float* q;
@@ -868,15 +903,19 @@ struct DeltaHeadArgs {
     const float* decay;         // [tokens][H]
     const int* qo_indptr;
     const int* slots;
-    float* T;                   // [H][tokens][C]
-    float* BT;                  // [H][tokens][C]
-    float* PS;                  // [H][tokens][2]: P_t, dec(C, t)
+    float* rows;                // [pieces][G][2 C][D + 4]: the k rows, then the q rows; zeros past the end
+    float* mats;                // [pieces][H][C][GH_MROW]
     float* state;
     long long state_stride;
     long long state_offset;
     float* out;
     int H, G, D, VD, tokens;
+    int* error_word;
+    ConvAdvance conv;
 };
+
+// Pieces are numbered over the batch so that an entry's are consecutive: at most tokens / C + entries.
+__device__ __forceinline__ size_t gh_first_piece(int start, int e) { return (size_t)(start / GC_TOKENS + e); }
 
 // A block per (piece, entry, group of heads); thread (t, j) of 256 makes k_t . k_j and q_t . k_j,
 // then a warp a head: lane j the column j of T and of B T by forward substitution.
@@ -888,7 +927,7 @@ __global__ void __launch_bounds__(256) delta_head_pieces_kernel(DeltaHeadArgs a)
     float* qs = ks + C * LD;                     // [C][LD]
     float* kk = qs + C * LD;                     // [C][GH_LD] k_t . k_j
     float* qk = kk + C * GH_LD;                  // [C][GH_LD] q_t . k_j
-    float* per_warp = qk + C * GH_LD;            // [8 warps]{L, B [C][GH_LD], g, beta, prefix [C]}
+    float* per_warp = qk + C * GH_LD;            // [min(8, heads of the group)]{L, B [C][GH_LD], g, beta [C]}
     const int piece = blockIdx.x, e = blockIdx.y, grp = blockIdx.z;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const unsigned long long waited = pdl_wait();
@@ -911,6 +950,9 @@ __global__ void __launch_bounds__(256) delta_head_pieces_kernel(DeltaHeadArgs a)
         }
         *reinterpret_cast<float4*>(ks + t * LD + d) = kv;
         *reinterpret_cast<float4*>(qs + t * LD + d) = qv;
+        float* dst = a.rows + (((gh_first_piece(start, e) + piece) * a.G + grp) * 2 * C + t) * LD + d;
+        *reinterpret_cast<float4*>(dst) = kv;
+        *reinterpret_cast<float4*>(dst + C * LD) = qv;
     }
     __syncthreads();
     {
@@ -934,7 +976,7 @@ __global__ void __launch_bounds__(256) delta_head_pieces_kernel(DeltaHeadArgs a)
     float* B = L + C * GH_LD;
     float* gs = B + C * GH_LD;
     float* bs = gs + C;
-    for (int i = warp; i < per; i += 8) {
+    for (int i = warp; i < per && warp < 8; i += 8) {
         const int h = grp * per + i;
         if (lane < C) {
             const size_t o = (size_t)(start + base + lane) * a.H + h;
@@ -955,18 +997,21 @@ __global__ void __launch_bounds__(256) delta_head_pieces_kernel(DeltaHeadArgs a)
         for (int t = 0; t <= j; ++t) P *= gs[t];
         __syncwarp();
         if (lane < C) {
-            const size_t first = (size_t)h * a.tokens + start + base;
-            if (j < here) {
-                a.PS[(first + j) * 2] = P;
-                a.PS[(first + j) * 2 + 1] = dec;         // dec(C, j): a short piece's g are 1 past its end
-            }
-            float col[C];                                 // column j of (I + L)^-1
+            float* m = a.mats + ((gh_first_piece(start, e) + piece) * a.H + h) * C * GH_MROW;
+            m[j * GH_MROW + 2 * C] = P;
+            m[j * GH_MROW + 2 * C + 1] = dec;            // dec(C, j): a short piece's g are 1 past its end
+            float col[C];                                 // column j of (I + L)^-1, zero above j
 #pragma unroll
             for (int t = 0; t < C; ++t) {
                 float s = t == j ? 1.f : 0.f;
 #pragma unroll
-                for (int m = 0; m < t; ++m)
-                    if (m >= j) s = fmaf(-L[t * GH_LD + m], col[m], s);
+                for (int x = 0; x < t; x += 4) {
+                    float l[4];
+                    load4(L + t * GH_LD + x, l);
+#pragma unroll
+                    for (int w = 0; w < 4; ++w)
+                        if (x + w < t) s = fmaf(-l[w], col[x + w], s);
+                }
                 col[t] = s;
             }
             const float bj = bs[j];
@@ -974,264 +1019,288 @@ __global__ void __launch_bounds__(256) delta_head_pieces_kernel(DeltaHeadArgs a)
             for (int t = 0; t < C; ++t) {
                 float s = 0.f;
 #pragma unroll
-                for (int m = 0; m <= t; ++m)
-                    if (m >= j) s = fmaf(B[t * GH_LD + m], col[m], s);
-                if (t < here) {
-                    a.T[(first + t) * C + j] = t >= j ? col[t] * bj : 0.f;
-                    a.BT[(first + t) * C + j] = s * bj;
+                for (int x = 0; x <= t; x += 4) {
+                    float bt[4];
+                    load4(B + t * GH_LD + x, bt);
+#pragma unroll
+                    for (int w = 0; w < 4; ++w)
+                        if (x + w <= t) s = fmaf(bt[w], col[x + w], s);
                 }
+                m[t * GH_MROW + j] = col[t] * bj;
+                m[t * GH_MROW + C + j] = s * bj;
             }
         }
         __syncwarp();
     }
 }
 
-// Two floats multiplied and added at once.
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 gh_fma2(f32x2 a, f32x2 b, f32x2 c) {
-    f32x2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
+// A block owns COLS (8 or 16) value columns of one head of one entry.  Per piece, all as small matrix
+// products in registers: [r; p] = [k; q] S0 (32 rows x COLS columns, each warp over a quarter of D, a
+// thread 4 rows x COLS / 4 columns), the warps' shares met in shared memory; c, then u = T c and o by
+// thread (t, COLS / 8 columns); S = P_C S0 + (dec k)^T u by a thread that keeps its part of S in registers and
+// leaves a copy, a column a row, in shared memory for the next piece's products.
+__device__ __forceinline__ void gh_load(const float* p, float (&v)[1]) { v[0] = p[0]; }
+__device__ __forceinline__ void gh_load(const float* p, float (&v)[2]) {
+    const float2 a = *reinterpret_cast<const float2*>(p);
+    v[0] = a.x; v[1] = a.y;
 }
-__device__ __forceinline__ f32x2 gh_pack(float lo, float hi) {
-    f32x2 d;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-    return d;
+__device__ __forceinline__ void gh_load(const float* p, float (&v)[4]) { load4(p, v); }
+__device__ __forceinline__ void gh_store(float* p, const float (&v)[1]) { p[0] = v[0]; }
+__device__ __forceinline__ void gh_store(float* p, const float (&v)[2]) {
+    *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
 }
-__device__ __forceinline__ float gh_both(f32x2 v) {
-    float lo, hi;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-    return lo + hi;
+__device__ __forceinline__ void gh_bulk(float* dst, const float* src, uint32_t bytes, uint32_t bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 ::"r"(tc_smem(dst)), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
-// A warp owns NC value columns of one head of one entry; a column's D = 32 R rows lie on the lanes,
-// R consecutive rows a lane.  Per piece: the columns go to shared memory; lane (t, half) takes
-// token t's products with all columns over one half of the rows (every key and query value it reads
-// meets NC columns); c goes round through shared memory, the lower lanes make u_t = (T c)_t, the
-// upper o_t; then the new columns.
-template <int R, int NC>
-__global__ void __launch_bounds__(GH_WARPS * 32) delta_head_scan_kernel(DeltaHeadArgs a) {
+template <int D, int COLS>
+__global__ void __launch_bounds__(GH_THREADS, 2) delta_head_scan_kernel(DeltaHeadArgs a) {
     extern __shared__ __align__(16) float sm[];
-    constexpr int C = GC_TOKENS, D = 32 * R, LD = D + 4, COLS = GH_WARPS * NC;
-    constexpr int per_buf = 2 * C * LD + 2 * C * GH_LD + C * COLS + 2 * C;
-    static_assert(per_buf % 4 == 0, "the second buffer starts on a 16-byte boundary");
-    constexpr int per_warp = NC * D + NC * C + 2 * C * NC;
+    constexpr int C = GC_TOKENS, LD = D + 4, WARPS = GH_THREADS / 32;
+    constexpr int per_buf = 2 * C * LD + C * GH_MROW;
+    constexpr int PJ = COLS / 4;                             // columns a thread takes of [r; p]
+    constexpr int CT = D >= 96 ? PJ : (D == 64 || PJ < 4 ? PJ / 2 : 1);      // and keeps of S
+    constexpr int TN = COLS / 8;                             // and makes of u and o
+    constexpr int DT = D > 128 ? D / 128 : 1;                // groups of 4 rows it keeps
+    constexpr int DG = D / 4 / DT;                           // row groups that lie on threads
+    constexpr int PLD = COLS + 4;
+    float* cols = sm + 2 * per_buf;              // [COLS][LD] S0, a column a row
+    float* part = cols + COLS * LD;              // [WARPS][2 C][PLD] shares of r and p
+    float* cs = part + WARPS * 2 * C * PLD;      // [C][COLS]
+    float* us = cs + C * COLS;                   // [C][COLS] dec(C, t) u_t
+    __shared__ __align__(8) unsigned long long full[2];
     const int e = blockIdx.x, h = blockIdx.y;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int col0 = blockIdx.z * COLS;
-    float* mine = sm + 2 * per_buf + warp * per_warp;
-    float* cols = mine;                          // [NC][D] the columns at a piece's start
-    float* cs = cols + NC * D;                   // [NC][C]
-    float* us = cs + NC * C;                     // [C][NC][2] dec(C, t) u_t, each number twice
     const unsigned long long waited = pdl_wait();
-    const float* q = pdl_after(a.q, waited);
-    const float* k = pdl_after(a.k, waited);
     const float* v = pdl_after(a.v, waited);
-    const float* T = pdl_after((const float*)a.T, waited);
-    const float* BT = pdl_after((const float*)a.BT, waited);
-    const float* PS = pdl_after((const float*)a.PS, waited);
+    const float* rows = pdl_after((const float*)a.rows, waited);
+    const float* mats = pdl_after((const float*)a.mats, waited);
     float* state = pdl_after(a.state, waited);
     const int start = a.qo_indptr[e], n = a.qo_indptr[e + 1] - start;
     if (n <= 0) return;
-    const int qkw = a.G * D, vv = a.H * a.VD, grp = h / (a.H / a.G);
-    const int ncols = min(COLS, a.VD - col0);
+    const int vv = a.H * a.VD, grp = h / (a.H / a.G);
+    const size_t first = gh_first_piece(start, e);
 
-    auto fetch = [&](int buf, int piece) {
-        const int base = piece * C;
-        const int here = min(C, n - base);
+    auto fetch = [&](int buf, int piece) {       // one thread; both copies complete on the buffer's barrier
+        const uint32_t bar = tc_smem(full + buf);
         float* dst = sm + buf * per_buf;
-        const size_t first = (size_t)h * a.tokens + start + base;
-        for (int i = tid; i < here * (D / 4); i += GH_WARPS * 32) {
-            const int t = i / (D / 4), d = (i - t * (D / 4)) * 4;
-            const size_t o = (size_t)(start + base + t) * qkw + (size_t)grp * D + d;
-            gd_copy16(dst + t * LD + d, k + o);
-            gd_copy16(dst + C * LD + t * LD + d, q + o);
-        }
-        float* m = dst + 2 * C * LD;
-        for (int i = tid; i < here * (C / 4); i += GH_WARPS * 32) {
-            const int t = i / (C / 4), j = (i - t * (C / 4)) * 4;
-            gd_copy16(m + t * GH_LD + j, T + (first + t) * C + j);
-            gd_copy16(m + C * GH_LD + t * GH_LD + j, BT + (first + t) * C + j);
-        }
-        float* vs = m + 2 * C * GH_LD;
-        for (int i = tid; i < here * COLS; i += GH_WARPS * 32) {
-            const int t = i / COLS, c = i - t * COLS;
-            if (c < ncols)
-                gd_copy4(vs + t * COLS + c, v + (size_t)(start + base + t) * vv + (size_t)h * a.VD + col0 + c);
-        }
-        for (int i = tid; i < here * 2; i += GH_WARPS * 32) gd_copy4(vs + C * COLS + i, PS + first * 2 + i);
+        mbar_expect_tx(bar, (uint32_t)(per_buf * sizeof(float)));
+        gh_bulk(dst, rows + ((first + piece) * a.G + grp) * 2 * C * LD, 2 * C * LD * sizeof(float), bar);
+        gh_bulk(dst + 2 * C * LD, mats + ((first + piece) * a.H + h) * C * GH_MROW, C * GH_MROW * sizeof(float), bar);
     };
 
-    // what no copy writes (columns past the last, rows past a short piece) reads as finite numbers
-    for (int i = tid; i < 2 * per_buf; i += GH_WARPS * 32) sm[i] = 0.f;
-    __syncthreads();
     const int pieces = (n + C - 1) / C;
-    fetch(0, 0);
-    cp_async_commit();
-    float* s_cols = state + (size_t)a.slots[e] * a.state_stride + a.state_offset +
-                    ((size_t)h * a.VD + col0 + warp * NC) * D;
-    float s[NC][R];
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-        if (warp * NC + c < ncols) {
-            gc_load<R>(s_cols + (size_t)c * D + lane * R, s[c]);
-        } else {
-#pragma unroll
-            for (int i = 0; i < R; ++i) s[c][i] = 0.f;
-        }
+    if (tid == 0) {
+        mbar_init(tc_smem(full), 1);
+        mbar_init(tc_smem(full + 1), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        fetch(0, 0);
     }
-    const int t = lane & 15, half = lane >> 4;
+    __syncthreads();
+    // the thread's part of S: rows 4 (dg + DG x) .. + 3, columns CT cg .. (lanes: 8 row groups x 4
+    // column groups)
+    const int cg = (tid / 8) % (COLS / CT), dg = tid % 8 + (tid / 8 / (COLS / CT)) * 8;
+    const bool keeps = dg < DG;
+    float* s_head = state + (size_t)a.slots[e] * a.state_stride + a.state_offset +
+                    ((size_t)h * a.VD + col0) * D;
+    float s[DT][CT][4];
+#pragma unroll
+    for (int x = 0; x < DT; ++x)
+#pragma unroll
+        for (int c = 0; c < CT; ++c) {
+            s[x][c][0] = s[x][c][1] = s[x][c][2] = s[x][c][3] = 0.f;
+            if (keeps) {
+                const int col = cg * CT + c, d = (dg + DG * x) * 4;
+                if (col0 + col < a.VD) load4(s_head + (size_t)col * D + d, s[x][c]);
+                store4(cols + col * LD + d, s[x][c]);
+            }
+        }
+    // thread (token t, columns tc .. tc + TN - 1) between the products
+    const int t = tid / 8, tc = tid % 8 * TN;
+    float v_next[TN];
+#pragma unroll
+    for (int x = 0; x < TN; ++x) v_next[x] = 0.f;
+    auto ahead = [&](int piece) {                // the values the thread itself needs of a piece
+        const int at = piece * C + t;
+        if (at < n) {
+            const float* src = v + (size_t)(start + at) * vv + (size_t)h * a.VD + col0 + tc;
+#pragma unroll
+            for (int x = 0; x < TN; ++x)
+                if (col0 + tc + x < a.VD) v_next[x] = src[x];
+        }
+    };
+    ahead(0);
+    const int tg = lane & 7, pg = lane >> 3;     // rows tg + 8 i of [k; q], columns pg + 4 j
     for (int piece = 0; piece < pieces; ++piece) {
         const int buf = piece & 1;
-        if (piece + 1 < pieces) fetch(buf ^ 1, piece + 1);
-        cp_async_commit();
-        cp_async_wait<1>();
+        if (!__all_sync(0xffffffffu, mbar_wait(tc_smem(full + buf), (piece >> 1) & 1))) {
+            if (lane == 0) atomicExch(a.error_word, GH_WAIT_CODE);
+            mbar_wait(tc_smem(full + buf), (piece >> 1) & 1);    // no copy in flight outlives the block
+            return;
+        }
+        __syncthreads();                         // the piece and S0 are here, the other buffer is free
+        float vt[TN];
 #pragma unroll
-        for (int c = 0; c < NC; ++c) gc_store<R>(cols + c * D + lane * R, s[c]);
-        __syncthreads();
+        for (int x = 0; x < TN; ++x) vt[x] = v_next[x];
+        if (piece + 1 < pieces) {
+            if (tid == 0) fetch(buf ^ 1, piece + 1);
+            ahead(piece + 1);
+        }
         const int here = min(C, n - piece * C);
-        const float* ks = sm + buf * per_buf;
-        const float* qs = ks + C * LD;
-        const float* ms = qs + C * LD;
-        const float* vs = ms + 2 * C * GH_LD;
-        const float* ps = vs + C * COLS;
-        f32x2 r2[NC], p2[NC];
-#pragma unroll
-        for (int c = 0; c < NC; ++c) r2[c] = p2[c] = 0ull;
+        const float* ks = sm + buf * per_buf;    // (the q rows follow the k rows)
+        const float* ms = ks + 2 * C * LD;
+        const float P = ms[t * GH_MROW + 2 * C], dec = ms[t * GH_MROW + 2 * C + 1];
         {
-            const ulonglong2* kr = reinterpret_cast<const ulonglong2*>(ks + t * LD + half * (D / 2));
-            const ulonglong2* qr = reinterpret_cast<const ulonglong2*>(qs + t * LD + half * (D / 2));
-            const ulonglong2* sr = reinterpret_cast<const ulonglong2*>(cols + half * (D / 2));
+            float acc[4][PJ];
 #pragma unroll
-            for (int i = 0; i < D / 8; ++i) {
-                const ulonglong2 k4 = kr[i], q4 = qr[i];
+            for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int c = 0; c < NC; ++c) {
-                    const ulonglong2 s4 = sr[c * (D / 4) + i];
-                    r2[c] = gh_fma2(k4.x, s4.x, r2[c]);
-                    p2[c] = gh_fma2(q4.x, s4.x, p2[c]);
-                    r2[c] = gh_fma2(k4.y, s4.y, r2[c]);
-                    p2[c] = gh_fma2(q4.y, s4.y, p2[c]);
-                }
+                for (int j = 0; j < PJ; ++j) acc[i][j] = 0.f;
+            const float* rowp = ks + tg * LD + warp * (D / WARPS);
+            const float* colp = cols + pg * LD + warp * (D / WARPS);
+#pragma unroll
+            for (int d = 0; d < D / WARPS; d += 4) {
+                float rv[4][4], cv[PJ][4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) load4(rowp + 8 * i * LD + d, rv[i]);
+#pragma unroll
+                for (int j = 0; j < PJ; ++j) load4(colp + 4 * j * LD + d, cv[j]);
+#pragma unroll
+                for (int w = 0; w < 4; ++w)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+#pragma unroll
+                        for (int j = 0; j < PJ; ++j) acc[i][j] = fmaf(rv[i][w], cv[j][w], acc[i][j]);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < PJ; ++j)
+                    part[(warp * 2 * C + tg + 8 * i) * PLD + pg + 4 * j] = acc[i][j];
+        }
+        __syncthreads();
+        float r[TN], p[TN];
+#pragma unroll
+        for (int x = 0; x < TN; ++x) r[x] = p[x] = 0.f;
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) {
+            float rs[TN], ps[TN];
+            gh_load(part + (w * 2 * C + t) * PLD + tc, rs);
+            gh_load(part + (w * 2 * C + C + t) * PLD + tc, ps);
+#pragma unroll
+            for (int x = 0; x < TN; ++x) {
+                r[x] += rs[x];
+                p[x] += ps[x];
             }
         }
-        const float P = ps[2 * t], dec = ps[2 * t + 1];
-        float o[NC];
+        // (a token past the piece has c = 0: its row and column of T and B T are not used)
+        float ct[TN];
 #pragma unroll
-        for (int c = 0; c < NC; ++c) {
-            float r = gh_both(r2[c]), p = gh_both(p2[c]);
-            r += __shfl_xor_sync(0xffffffffu, r, 16);
-            p += __shfl_xor_sync(0xffffffffu, p, 16);
-            o[c] = half ? P * p : 0.f;
-            // (a token past the piece has c = 0: its row and column of T and B T are not used)
-            if (half == 0) cs[c * C + t] = t < here ? vs[t * COLS + warp * NC + c] - P * r : 0.f;
-        }
-        __syncwarp();
+        for (int x = 0; x < TN; ++x) ct[x] = t < here ? fmaf(-P, r[x], vt[x]) : 0.f;
+        gh_store(cs + t * COLS + tc, ct);
+        __syncthreads();
         {
-            const float4* row = reinterpret_cast<const float4*>(ms + half * C * GH_LD + t * GH_LD);
-            const float4* cv = reinterpret_cast<const float4*>(cs);
+            float u[TN], o[TN];
 #pragma unroll
-            for (int i = 0; i < C / 4; ++i) {
-                const float4 m4 = row[i];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) {
-                    const float4 c4 = cv[c * (C / 4) + i];
-                    o[c] = fmaf(m4.x, c4.x, o[c]);
-                    o[c] = fmaf(m4.y, c4.y, o[c]);
-                    o[c] = fmaf(m4.z, c4.z, o[c]);
-                    o[c] = fmaf(m4.w, c4.w, o[c]);
-                }
+            for (int x = 0; x < TN; ++x) {
+                u[x] = 0.f;
+                o[x] = P * p[x];
             }
-        }
-        if (half == 0) {                         // o holds u_t here
+            const float* trow = ms + t * GH_MROW;
+            const float* brow = trow + C;
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                const float u = t < here ? dec * o[c] : 0.f;
-                *reinterpret_cast<float2*>(us + (t * NC + c) * 2) = make_float2(u, u);
-            }
-        } else if (t < here) {
-            float* dst = a.out + (size_t)(start + piece * C + t) * vv + (size_t)h * a.VD + col0 + warp * NC;
+            for (int i = 0; i < C; i += 4) {
+                float t4[4], b4[4];
+                load4(trow + i, t4);
+                load4(brow + i, b4);
 #pragma unroll
-            for (int c = 0; c < NC; ++c)
-                if (warp * NC + c < ncols) dst[c] = o[c];
-        }
-        __syncwarp();
-        const float PC = ps[2 * (here - 1)];
-        if constexpr (R >= 2) {
-            f32x2 s2[NC][R / 2];
-            const f32x2 pc2 = gh_pack(PC, PC);
+                for (int w = 0; w < 4; ++w) {
+                    float c[TN];
+                    gh_load(cs + (i + w) * COLS + tc, c);
 #pragma unroll
-            for (int c = 0; c < NC; ++c)
-#pragma unroll
-                for (int i = 0; i < R / 2; ++i)
-                    s2[c][i] = gh_fma2(gh_pack(s[c][2 * i], s[c][2 * i + 1]), pc2, 0ull);
-#pragma unroll 4
-            for (int j = 0; j < C; ++j) {
-                f32x2 kv[R / 2];
-                if constexpr (R == 2) {
-                    kv[0] = *reinterpret_cast<const f32x2*>(ks + j * LD + lane * R);
-                } else {
-#pragma unroll
-                    for (int i = 0; i < R / 4; ++i) {
-                        const ulonglong2 k4 = reinterpret_cast<const ulonglong2*>(ks + j * LD + lane * R)[i];
-                        kv[2 * i] = k4.x;
-                        kv[2 * i + 1] = k4.y;
-                    }
-                }
-#pragma unroll
-                for (int c = 0; c < NC; c += 2) {
-                    const ulonglong2 u2 = *reinterpret_cast<const ulonglong2*>(us + (j * NC + c) * 2);
-#pragma unroll
-                    for (int i = 0; i < R / 2; ++i) {
-                        s2[c][i] = gh_fma2(kv[i], u2.x, s2[c][i]);
-                        s2[c + 1][i] = gh_fma2(kv[i], u2.y, s2[c + 1][i]);
+                    for (int x = 0; x < TN; ++x) {
+                        u[x] = fmaf(t4[w], c[x], u[x]);
+                        o[x] = fmaf(b4[w], c[x], o[x]);
                     }
                 }
             }
 #pragma unroll
-            for (int c = 0; c < NC; ++c)
+            for (int x = 0; x < TN; ++x) u[x] = t < here ? dec * u[x] : 0.f;
+            gh_store(us + t * COLS + tc, u);
+            if (t < here) {
+                float* dst = a.out + (size_t)(start + piece * C + t) * vv + (size_t)h * a.VD + col0 + tc;
 #pragma unroll
-                for (int i = 0; i < R / 2; ++i)
-                    asm("mov.b64 {%0, %1}, %2;" : "=f"(s[c][2 * i]), "=f"(s[c][2 * i + 1]) : "l"(s2[c][i]));
-        } else {
-#pragma unroll
-            for (int c = 0; c < NC; ++c) s[c][0] *= PC;
-#pragma unroll 4
-            for (int j = 0; j < C; ++j) {
-                const float kv = ks[j * LD + lane];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) s[c][0] = fmaf(kv, us[(j * NC + c) * 2], s[c][0]);
+                for (int x = 0; x < TN; ++x)
+                    if (col0 + tc + x < a.VD) dst[x] = o[x];
             }
         }
-        __syncthreads();                       // the buffer is free for the piece after next
+        __syncthreads();
+        if (keeps) {
+            const float pc = ms[(here - 1) * GH_MROW + 2 * C];
+#pragma unroll
+            for (int x = 0; x < DT; ++x)
+#pragma unroll
+                for (int c = 0; c < CT; ++c)
+#pragma unroll
+                    for (int w = 0; w < 4; ++w) s[x][c][w] *= pc;
+#pragma unroll
+            for (int j = 0; j < C; ++j) {
+                float u[CT];
+                gh_load(us + j * COLS + cg * CT, u);
+#pragma unroll
+                for (int x = 0; x < DT; ++x) {
+                    float kv[4];
+                    load4(ks + j * LD + (dg + DG * x) * 4, kv);
+#pragma unroll
+                    for (int c = 0; c < CT; ++c)
+#pragma unroll
+                        for (int w = 0; w < 4; ++w) s[x][c][w] = fmaf(kv[w], u[c], s[x][c][w]);
+                }
+            }
+#pragma unroll
+            for (int x = 0; x < DT; ++x)
+#pragma unroll
+                for (int c = 0; c < CT; ++c) store4(cols + (cg * CT + c) * LD + (dg + DG * x) * 4, s[x][c]);
+        }
     }
-    cp_async_wait<0>();
+    if (keeps) {
 #pragma unroll
-    for (int c = 0; c < NC; ++c)
-        if (warp * NC + c < ncols) gc_store<R>(s_cols + (size_t)c * D + lane * R, s[c]);
+        for (int x = 0; x < DT; ++x)
+#pragma unroll
+            for (int c = 0; c < CT; ++c)
+                if (col0 + cg * CT + c < a.VD)
+                    store4(s_head + (size_t)(cg * CT + c) * D + (dg + DG * x) * 4, s[x][c]);
+    }
+    gd_advance_conv(a.conv, waited, state + (size_t)a.slots[e] * a.state_stride, start, n, h, a.H);
 }
 
-// The scan in pieces with one decay a head (`decay` [tokens][H]), for key sizes of 32, 64, 128 or
-// 256: `work` holds tokens * H * (2 * 16 + 2) floats.  Returns 0, a CUDA error code, or -1 when the
+// The scan in pieces with one decay a head (`decay` [tokens][H]), for key sizes of 32, 64, 96, 128 or
+// 256: `work` holds (tokens / 16 + entries) * (G * 32 * (D + 4) + H * 16 * 36) floats.  Returns 0, a CUDA error code, or -1 when the
 // shape is refused.
 MSTAR_API int mstar_delta_scan_head_pieces(const float* q, const float* k, const float* v,
                                            const float* beta, const float* decay,
                                            const int* qo_indptr, const int* slots, float* state,
                                            long long state_stride, long long state_offset, float* out,
                                            float* work, int tokens, int entries, int max_q_len, int H,
-                                           int G, int D, int VD, void* stream) {
+                                           int G, int D, int VD, int* error_word, const float* conv_raw,
+                                           int conv_ld, int channels, int taps, void* stream) {
     if (entries <= 0 || tokens <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || VD <= 0) return -1;
-    if (D != 32 && D != 64 && D != 128 && D != 256) return -1;
+    if (D != 32 && D != 64 && D != 96 && D != 128 && D != 256) return -1;
     if (H > 65535 || entries > 65535 || (state_offset % 4) != 0 || (state_stride % 4) != 0) return -1;
-    if ((uintptr_t)q % 16 || (uintptr_t)k % 16 || (uintptr_t)work % 16 || (uintptr_t)state % 16) return -1;
+    if ((uintptr_t)q % 16 || (uintptr_t)k % 16 || (uintptr_t)work % 16 || (uintptr_t)state % 16 || !error_word)
+        return -1;
     const int max_pieces = (max_q_len + GC_TOKENS - 1) / GC_TOKENS;
-    const size_t th = (size_t)tokens * H;
-    DeltaHeadArgs a{q, k, v, beta, decay, qo_indptr, slots, work, work + th * GC_TOKENS,
-                    work + 2 * th * GC_TOKENS, state, state_stride, state_offset, out, H, G, D, VD, tokens};
+    const size_t most = (size_t)(tokens / GC_TOKENS + entries);
+    DeltaHeadArgs a{q, k, v, beta, decay, qo_indptr, slots, work, work + most * G * 2 * GC_TOKENS * (D + 4), state, state_stride, state_offset, out, H, G, D, VD, tokens,
+                    error_word, {taps > 1 ? conv_raw : nullptr, conv_ld, channels, taps}};
     cudaStream_t s = (cudaStream_t)stream;
+    // a warp a head in the second half of the first kernel: eight at most, as many as a group has
+    const int per = H / G, warps = per < 8 ? per : 8;
     const size_t smem1 = (2 * (size_t)GC_TOKENS * (D + 4) + 2 * GC_TOKENS * GH_LD +
-                          8 * (2 * GC_TOKENS * GH_LD + 2 * GC_TOKENS)) * sizeof(float);
+                          warps * (2 * GC_TOKENS * GH_LD + 2 * GC_TOKENS)) * sizeof(float);
     if (smem1 > 48 * 1024) {
         static size_t configured = 0;
         if (smem1 > configured) {
@@ -1243,33 +1312,31 @@ MSTAR_API int mstar_delta_scan_head_pieces(const float* q, const float* k, const
     mstar_launch(delta_head_pieces_kernel, dim3(max_pieces, entries, G), dim3(256), smem1, s, a);
     int code = launch_status();
     if (code != 0) return code;
-    // four columns a warp where that still gives half the SMs a block, else two
-    const int nc = (long long)entries * H * ((VD + 4 * GH_WARPS - 1) / (4 * GH_WARPS)) * 2 >=
-                           device_sm_count() ? 4 : 2;
-    const int cols = nc * GH_WARPS;
-    const size_t smem2 = ((size_t)2 * (2 * GC_TOKENS * (D + 4) + 2 * GC_TOKENS * GH_LD +
-                                       GC_TOKENS * cols + 2 * GC_TOKENS) +
-                          (size_t)GH_WARPS * (nc * D + nc * GC_TOKENS + 2 * GC_TOKENS * nc)) * sizeof(float);
+    // 16 columns a block where that gives most SMs a block, else 8
+    const int cols = (long long)entries * H * ((VD + 15) / 16) * 4 >= 3LL * device_sm_count() ? 16 : 8;
+    const size_t smem2 = ((size_t)2 * (2 * GC_TOKENS * (D + 4) + GC_TOKENS * GH_MROW) + cols * (D + 4) +
+                          (GH_THREADS / 32) * 2 * GC_TOKENS * (cols + 4) + 2 * GC_TOKENS * cols) * sizeof(float);
     dim3 grid(entries, H, (VD + cols - 1) / cols);
     if (grid.z > 65535) return -1;
-#define GO1(RR, NN)                                                                               \
+#define GO1(DD, CC)                                                                               \
     do {                                                                                          \
         static size_t configured = 0;                                                             \
         if (smem2 > 48 * 1024 && smem2 > configured) {                                            \
-            cudaFuncSetAttribute(delta_head_scan_kernel<RR, NN>,                                  \
+            cudaFuncSetAttribute(delta_head_scan_kernel<DD, CC>,                                  \
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);        \
             configured = smem2;                                                                   \
         }                                                                                         \
-        mstar_launch((delta_head_scan_kernel<RR, NN>), grid, dim3(GH_WARPS * 32), smem2, s, a);   \
+        mstar_launch((delta_head_scan_kernel<DD, CC>), grid, dim3(GH_THREADS), smem2, s, a);      \
     } while (0)
-#define GO(RR)                                                                                    \
+#define GO(DD)                                                                                    \
     do {                                                                                          \
-        if (nc == 4) GO1(RR, 4); else GO1(RR, 2);                                                 \
+        if (cols == 16) GO1(DD, 16); else GO1(DD, 8);                                             \
     } while (0)
-    if (D == 32) GO(1);
-    else if (D == 64) GO(2);
-    else if (D == 128) GO(4);
-    else GO(8);
+    if (D == 32) GO(32);
+    else if (D == 64) GO(64);
+    else if (D == 96) GO(96);
+    else if (D == 128) GO(128);
+    else GO(256);
 #undef GO
 #undef GO1
     return launch_status();

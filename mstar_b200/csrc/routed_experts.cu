@@ -34,25 +34,21 @@
 #define RT_PER_LANE 32
 #define RT_MAX_GROUPS 1024
 
-// The largest (value, index) of a warp's lanes, the lower index winning a tie; an index of
-// 0x7fffffff is no candidate.
-__device__ __forceinline__ void rt_warp_best(float& bz, int& be) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float oz = __shfl_xor_sync(0xffffffffu, bz, o);
-        const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-        if (oe != 0x7fffffff && (be == 0x7fffffff || oz > bz || (oz == bz && oe < be))) {
-            bz = oz;
-            be = oe;
-        }
-    }
+// The index of the largest value of a warp's lanes (a lane offers value bz at index be), the lower
+// index winning a tie; an index of 0x7fffffff is no candidate.  Two integer reductions on keys that
+// order as the floats do.
+__device__ __forceinline__ int rt_warp_best(float bz, int be) {
+    const unsigned bits = __float_as_uint(bz + 0.f);                 // (-0 and 0 are equal)
+    const unsigned key = be == 0x7fffffff ? 0u : (bits & 0x80000000u) ? ~bits : bits | 0x80000000u;
+    const unsigned most = __reduce_max_sync(0xffffffffu, key);
+    return (int)__reduce_min_sync(0xffffffffu, key == most ? (unsigned)be : 0x7fffffffu);
 }
 
 // The choice where it cannot be read off the logits alone: choice scores s + bias are made once
 // and kept in shared memory, and, with groups, the experts of all but the best `keep` groups are
 // closed.  A warp per token; the scores of a row lie at dynamic shared memory [warp][experts], the
 // groups' after all warps' scores ([warp][groups]).
-__global__ void route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ choice_bias,
+__global__ void route_choice_kernel(const float* __restrict__ logits, const float* __restrict__ choice_bias,
                                      int* __restrict__ chosen, float* __restrict__ weight, int tokens,
                                      int experts, int top, int softmax, int renormalize, int ld,
                                      int groups, int keep, float renorm_eps, float weight_scale) {
@@ -95,7 +91,7 @@ __global__ void route_grouped_kernel(const float* __restrict__ logits, const flo
                     bz = best[g];
                     be = g;
                 }
-            rt_warp_best(bz, be);
+            be = rt_warp_best(bz, be);
             if ((be & 31) == lane) open_groups |= 1u << (be >> 5);
         }
         // the mark of a kept group goes where every lane reads it
@@ -114,7 +110,7 @@ __global__ void route_grouped_kernel(const float* __restrict__ logits, const flo
                 bz = choice[e];
                 be = e;
             }
-        rt_warp_best(bz, be);
+        be = rt_warp_best(bz, be);
         if ((be & 31) == lane) closed |= 1u << (be >> 5);
         const float s = score(z[be]);
         total += s;
@@ -130,7 +126,7 @@ __global__ void route_grouped_kernel(const float* __restrict__ logits, const flo
     }
 }
 
-__global__ void route_topk_kernel(const float* __restrict__ logits, const float* __restrict__ choice_bias,
+__global__ void route_topk_kernel(const float* __restrict__ logits,
                                   int* __restrict__ chosen,
                                   float* __restrict__ weight, int tokens, int experts, int top,
                                   int softmax, int renormalize, int ld) {
@@ -156,25 +152,14 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, const float*
             const int e = lane + 32 * i;
             if (e >= experts) break;
             if (!((taken >> i) & 1u)) {
-                // scores are monotone in the logits; with a bias the choice needs the scores
-                float v = z[e];
-                if (choice_bias != nullptr)
-                    v = (softmax ? expf(v - zmax) / denom : 1.f / (1.f + expf(-v))) + choice_bias[e];
+                const float v = z[e];                 // scores are monotone in the logits
                 if (be == 0x7fffffff || v > bz) {
                     bz = v;
                     be = e;
                 }
             }
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float oz = __shfl_xor_sync(0xffffffffu, bz, o);
-            const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-            if (oe != 0x7fffffff && (be == 0x7fffffff || oz > bz || (oz == bz && oe < be))) {
-                bz = oz;
-                be = oe;
-            }
-        }
+        be = rt_warp_best(bz, be);
         if ((be & 31) == lane) taken |= 1u << (be >> 5);
         const float zb = z[be];
         const float s = softmax ? expf(zb - zmax) / denom : 1.f / (1.f + expf(-zb));
@@ -198,16 +183,16 @@ MSTAR_API int mstar_route_topk(const float* logits, const float* choice_bias, in
     if (groups > 0 && (groups > RT_MAX_GROUPS || experts % groups || keep <= 0 || keep > groups ||
                        top > experts / groups * keep))
         return -1;
-    if (groups > 0 || renorm_eps != 0.f || weight_scale != 1.f) {
+    if (groups > 0 || choice_bias != nullptr || renorm_eps != 0.f || weight_scale != 1.f) {
         // four warps' scores: at most 4 * (1,024 + 1,024) floats
         const size_t smem = sizeof(float) * 4 * (size_t)(experts + (groups > 0 ? groups : 0));
-        mstar_launch(route_grouped_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream,
+        mstar_launch(route_choice_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream,
                      logits, choice_bias, chosen, weight, tokens, experts, top, softmax, renormalize,
                      ld, groups, keep, renorm_eps, weight_scale);
         return launch_status();
     }
     mstar_launch(route_topk_kernel, dim3((tokens + 3) / 4), dim3(128), 0, (cudaStream_t)stream,
-                 logits, choice_bias, chosen, weight, tokens, experts, top, softmax, renormalize, ld);
+                 logits, chosen, weight, tokens, experts, top, softmax, renormalize, ld);
     return launch_status();
 }
 

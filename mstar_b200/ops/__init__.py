@@ -589,8 +589,8 @@ _tc_error_words: dict = {}
 def tcgen05_error_word(device) -> torch.Tensor:
     """Device int32 that a kernel with bounded mbarrier waits sets when one of them ran out:
     1-3 tcgen05 GEMM (producer, MMA issuer, epilogue), 4 decode attention copies, 6-12 tcgen05
-    prefill attention, 13-14 bulk-copy small-M GEMM, 15-17 swapped-operand tcgen05 GEMM; zero
-    otherwise."""
+    prefill attention, 13-14 bulk-copy small-M GEMM, 15-17 swapped-operand tcgen05 GEMM, 18
+    delta-rule scan in pieces; zero otherwise."""
     key = torch.device(device).index or 0
     if key not in _tc_error_words:
         _tc_error_words[key] = torch.zeros(1, dtype=torch.int32, device=device)
@@ -609,6 +609,7 @@ WAIT_CODES = {
 WAIT_CODES.update({15: "swapped-operand tcgen05 GEMM: the producer waited for a free stage",
                    16: "swapped-operand tcgen05 GEMM: the MMA issuer waited for operand tiles",
                    17: "swapped-operand tcgen05 GEMM: the epilogue waited for the accumulator"})
+WAIT_CODES[18] = "delta-rule scan in pieces: a wait for a piece's rows"
 WAIT_CODES.update({c: "tcgen05 prefill attention: a wait on one of its barriers ran out"
                    for c in range(6, 13)})
 
@@ -1758,7 +1759,7 @@ def delta_prepare(proj: torch.Tensor, conv_w: torch.Tensor, a_proj: torch.Tensor
     SiLU on the q, k and v channels (``conv_w`` [channels, taps]; rows before a portion from
     ``state``), unit q (times ``dim ** -0.5``) and k per head, ``beta = sigmoid(b)``, and the
     decays ``exp(-a_exp[h] * softplus(a_proj + dt_bias))``.  Returns float (q, k, v, beta,
-    decay).  ``conv_state_advance`` moves the slot's rows on afterwards."""
+    decay).  ``delta_scan`` (with ``conv_rows``) moves the slot's rows on afterwards."""
     _need_cuda(proj, conv_w, a_proj, dt_bias, a_exp, token_req, qo_indptr, slots, state)
     tokens = proj.shape[0]
     qk, vv = kv_heads * dim, heads * vdim
@@ -1796,11 +1797,12 @@ def delta_prepare(proj: torch.Tensor, conv_w: torch.Tensor, a_proj: torch.Tensor
 DELTA_PIECE = 16            # tokens of a piece of the delta-rule scan
 DELTA_PIECES_FROM = 64      # entries of this many tokens or more are scanned in pieces
 DELTA_PIECES_DIMS = (32, 64, 128, 256)     # key sizes the scan in pieces takes
+DELTA_HEAD_PIECES_DIMS = (32, 64, 96, 128, 256)    # with one decay a head
 
 
 def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entries: int,
                heads: int, kv_heads: int, dim: int, vdim: int, taps: int,
-               max_q_len: int = 1 << 30) -> torch.Tensor:
+               max_q_len: int = 1 << 30, conv_rows=None) -> torch.Tensor:
     """The gated delta rule over the tokens of ``entries`` batch entries, each continuing the
     matrix in its slot (updated in place).  ``max_q_len``: the longest entry (a bound will do;
     short entries stage fewer tokens at a time).  Returns float [tokens, heads * vdim].
@@ -1810,7 +1812,10 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
     queries, the keys' products among themselves) is made for all pieces side by side, and
     the chain from token to token shrinks to a scalar a token (MSTAR_DELTA_PIECES=0: never;
     1: always).  ``decay`` [tokens, heads] is one decay a head: the chain inside a piece then
-    becomes a small triangular matrix made ahead."""
+    becomes a small triangular matrix made ahead.
+
+    ``conv_rows``: the projected rows ``delta_prepare`` read; the slots' convolution inputs then
+    move on in the same launch (else ``conv_state_advance`` does that)."""
     _need_cuda(q, k, v, beta, decay, qo_indptr, slots, state)
     for t in (q, k, v, beta, decay):
         assert t.dtype == torch.float32 and t.is_contiguous()
@@ -1819,21 +1824,30 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
     head_decay = tuple(decay.shape) == (tokens, heads) and dim > 1
     assert head_decay or tuple(decay.shape) == (tokens, heads * dim)
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=q.device)
-    offset = (taps - 1) * (2 * kv_heads * dim + heads * vdim)
+    channels = 2 * kv_heads * dim + heads * vdim
+    offset = (taps - 1) * channels
+    conv = (0, 0, 0, 0)
+    if conv_rows is not None and taps > 1:
+        _need_cuda(conv_rows)
+        assert conv_rows.dtype == torch.float32 and conv_rows.stride(1) == 1
+        assert conv_rows.shape[0] == tokens and conv_rows.shape[1] >= channels
+        conv = (conv_rows.data_ptr(), conv_rows.stride(0), channels, taps)
     longest = int(min(max_q_len, tokens))
     forced = os.environ.get("MSTAR_DELTA_PIECES")
     pieces = (forced == "1" or (forced != "0" and longest >= DELTA_PIECES_FROM))
-    if (pieces and dim in DELTA_PIECES_DIMS and tokens > 0 and offset % 4 == 0
+    if (pieces and dim in (DELTA_HEAD_PIECES_DIMS if head_decay else DELTA_PIECES_DIMS) and tokens > 0 and offset % 4 == 0
             and state.stride(0) % 4 == 0):
         max_pieces = -(-longest // DELTA_PIECE)
         if head_decay:
-            work = torch.empty(tokens * heads * (2 * DELTA_PIECE + 2), dtype=torch.float32,
+            per_piece = (kv_heads * 2 * DELTA_PIECE * (dim + 4)
+                         + heads * DELTA_PIECE * (2 * DELTA_PIECE + 4))
+            work = torch.empty((tokens // DELTA_PIECE + entries) * per_piece, dtype=torch.float32,
                                device=q.device)
             code = lib.get("gated_delta").mstar_delta_scan_head_pieces(
                 q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), decay.data_ptr(),
                 qo_indptr.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0), offset,
                 out.data_ptr(), work.data_ptr(), tokens, entries, longest, heads, kv_heads, dim,
-                vdim, _stream())
+                vdim, tcgen05_error_word(q.device).data_ptr(), *conv, _stream())
             if code == -1:
                 raise KernelError(f"delta-rule scan in pieces refuses heads={heads}, "
                                   f"kv_heads={kv_heads}, dim={dim}")
@@ -1847,7 +1861,7 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
             q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), decay.data_ptr(),
             qo_indptr.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0), offset,
             out.data_ptr(), work.data_ptr(), tokens, entries, longest, heads, kv_heads, dim, vdim,
-            _stream())
+            *conv, _stream())
         if code == -1:
             raise KernelError(f"delta-rule scan in pieces refuses heads={heads}, "
                               f"kv_heads={kv_heads}, dim={dim}")
@@ -1858,7 +1872,7 @@ def delta_scan(q, k, v, beta, decay, qo_indptr, slots, state: torch.Tensor, entr
         q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), decay.data_ptr(),
         qo_indptr.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0), offset,
         out.data_ptr(), entries, int(min(max_q_len, 1 << 30)), heads, kv_heads, dim, vdim,
-        int(head_decay), _stream())
+        int(head_decay), *conv, _stream())
     if code == -1:
         raise KernelError(f"delta-rule scan refuses heads={heads}, kv_heads={kv_heads}, dim={dim} "
                           "(dim at most 512)")

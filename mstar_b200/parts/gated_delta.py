@@ -5,8 +5,8 @@ last inputs of its short convolutions live in a state slot.
 One product, with float output, gives ``[q | k | v | b | a1 | g1]``; two small products give
 the decay's pre-activation (``W_a2 a1``, float) and the output gate (``W_g2 g1``).  A kernel
 runs the convolutions with SiLU, makes q and k unit vectors, the write strengths and the
-decays (all float); a second moves the slot's convolution rows on; the scan walks each
-entry's tokens from the matrix in its slot; a last kernel norms each head's output, gates it
+decays (all float); the scan walks each entry's tokens from the matrix in its slot and moves
+the slot's convolution rows on; a last kernel norms each head's output, gates it
 and hands it to the output product.  With one decay a head and a gate that is a single product
 the first product gives everything, ``[q | k | v | b | a | g]``.  A prompt portion, a decoded token and any mix are the
 same launches.
@@ -84,10 +84,8 @@ class GatedDelta:
         q, k, v, beta, decay = ops.delta_prepare(
             proj, self.conv_w, a_proj, self.dt_bias, self.a_exp, ctx.token_req, ctx.qo_indptr,
             ctx.slots, cache.state, H, G, D, VD, s.conv, s.unit_eps)
-        ops.conv_state_advance(proj, channels, s.conv, ctx.qo_indptr, ctx.slots, cache.state,
-                               ctx.num_entries)
         o = ops.delta_scan(q, k, v, beta, decay, ctx.qo_indptr, ctx.slots, cache.state,
-                           ctx.num_entries, H, G, D, VD, s.conv, max_q_len=ctx.max_q_len)
+                           ctx.num_entries, H, G, D, VD, s.conv, max_q_len=ctx.max_q_len, conv_rows=proj)
         y = ops.delta_finish(o, gate, self.norm_weight, H, VD, s.norm_eps, self.runtime.dtype,
                              self.out_scale, s.gate_activation)
         return ops.linear(y, self.w_out, static_weights=True)

@@ -429,11 +429,10 @@ def test_delta_rule_with_one_decay_a_head(dtype, heads, kv_heads, dim, vdim, tap
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,taps",
                          [(4, 2, 24, 20, 3), (2, 1, 128, 40, 2), (2, 2, 200, 9, 1), (5, 1, 64, 64, 3),
                           (2, 2, 32, 12, 3), (2, 1, 256, 20, 2), (3, 1, 64, 7, 4), (24, 2, 32, 36, 4),
-                          (16, 4, 128, 128, 4)])
+                          (16, 4, 128, 128, 4), (3, 3, 96, 10, 4)])
 def test_delta_rule_long_portions_in_pieces(dtype, heads, kv_heads, dim, vdim, taps):
-    """A portion long enough to be scanned in pieces of 16 tokens (key sizes of 32, 64, 128 and 256,
-    two or four columns a warp; the others and a state that does not start on a 16-byte boundary
-    token by token), beside a short portion of another request in the same batch; then more
+    """A portion long enough to be scanned in pieces of 16 tokens (key sizes of 32, 64, 96, 128
+    and 256; the others and a state that does not start on a 16-byte boundary token by token), beside a short portion of another request in the same batch; then more
     tokens of both, a portion that is no multiple of 16 and a last one of a single token."""
     from mstar_b200 import ops
     from mstar_b200.parts import LayerCache
