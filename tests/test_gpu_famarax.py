@@ -202,7 +202,7 @@ ATTENTIONS = [
     (U.attention(4, 2, 128, 128, scale=0.19, softcap=9.0, window=None, rot_dims=128, base=7e4), 16),
     (U.attention(1, 1, 20, 20, scale=1.0, softcap=4.0, window=50, rot_dims=2, base=10.0), 8),
     (U.attention(5, 5, 96, 72, scale=0.25, window=17, rot_dims=0), 16),
-    (U.attention(8, 2, 64, 64, scale=0.1875, softcap=20.0, window=33, rot_dims=64), 16),
+    (U.attention(8, 2, 64, 64, scale=0.21, softcap=18.0, window=33, rot_dims=64), 16),
 ]
 
 
@@ -268,7 +268,7 @@ def marked_inputs(p, m, width, T, marked, queries, gain=6.0):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("window,page", [(96, 16), (97, 16), (64, 4), (130, 8), (16, 16)])
+@pytest.mark.parametrize("window,page", [(80, 16), (81, 16), (64, 4), (130, 8), (16, 16)])
 def test_edges_of_a_window(dtype, window, page):
     """A key that stands out is the oldest of one query's window and just outside the next
     query's: in one prompt, in portions cut at and around both, and decoded.  Inside, the output
@@ -538,7 +538,7 @@ def test_head_norm_and_silu_gate(dtype, vdim):
 
 # ------------------------------------------------------------------ experts
 @pytest.mark.parametrize("experts,top,groups,scale", [
-    (8, 3, (4, 2), 1.6), (6, 2, (2, 1), 0.8), (9, 4, (3, 2), 1.0), (5, 5, None, 2.0), (16, 4, (4, 3), 2.0),
+    (8, 3, (4, 2), 1.6), (6, 2, (2, 1), 0.8), (9, 4, (3, 2), 1.0), (5, 5, None, 2.0), (20, 4, (5, 3), 2.2),
     (64, 8, (32, 5), 1.5), (256, 8, (8, 4), 2.5), (1024, 16, (512, 9), 1.0), (40, 4, (1, 1), 0.5),
     (12, 3, (4, 1), 1.0), (1, 1, (1, 1), 3.0)])
 def test_choice_of_experts(experts, top, groups, scale):
